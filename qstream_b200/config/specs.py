@@ -51,6 +51,15 @@ class StreamNormSpec:
 
 
 @dataclass(frozen=True)
+class TanhNormSpec:
+    """The dynamic tanh in a norm's place: tanh(alpha x) * w + b with a scalar `alpha` and vectors w and b of `size`, no mean
+    and no variance.  It reads a residual stream in 32-bit and writes the engine's type."""
+    size: int
+    kind: str = "tanh_norm"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
 class RotaryHalfSpec:
     """Rotary position encoding on the first `rotary_dim` dims of a vector, element i paired with i + rotary_dim/2,
     angle position * f_i, f_i = base^(-2i / rotary_dim).  `scaling` (factor, original, fast, slow) rescales the
@@ -97,7 +106,7 @@ class AttentionSpec:
     `v_head_dim`: the values' head size where it differs from that of queries and keys.
     `score_scale`: the factor on q.k (default head_dim^-1/2).  `softcap` c > 0: scores
     become c tanh(s / c) before the softmax.  `gate`: the concatenated heads are multiplied
-    by sigmoid(W_g h) before the output projection.  `value_mix`: "first" keeps the layer's
+    by sigmoid(W_g h) before the output projection; "head": head h's output by sigmoid(W_g h)_h, W_g having one row per head.  `value_mix`: "first" keeps the layer's
     values for later layers of the same step, "blend" caches (1 - l) v + l v_first with its
     scalar tensor "value_mix" as l.
     `chunk` c > 0: a query sees only the keys of its own chunk of c positions; chunks tile the sequence from its first token (no window then).
@@ -127,7 +136,7 @@ class AttentionSpec:
     v_head_dim: Optional[int] = None
     score_scale: Optional[float] = None
     softcap: float = 0.0
-    gate: bool = False
+    gate: object = False                # False, True (a value per channel) or "head" (a value per head)
     value_mix: Optional[str] = None
     chunk: int = 0
     keep_first: int = 0
@@ -263,17 +272,75 @@ class GatedDeltaSpec:
 @dataclass(frozen=True)
 class PairMixerSpec:
     """Two mixers side by side that read the same input: left_scale * left(h) + right_scale * right(h).  Each keeps its
-    own cache entry (a schedule run names two)."""
+    own cache entry (a schedule run names two).  `norm_names` (the checkpoint names of two vectors of `width`): each
+    result is first divided by its root mean square over the width (`eps` inside the root), times its vector."""
     left: object
     right: object
     left_scale: float = 1.0
     right_scale: float = 1.0
     kind: str = "pair"
+    norm_names: Optional[Tuple[str, str]] = None
+    width: int = 0
+    eps: float = 0.0
 
     @property
     def names(self) -> Mapping[str, str]:
-        """The two mixers' tensors under "left.<name>" and "right.<name>"."""
-        return {**{"left." + k: v for k, v in self.left.names.items()}, **{"right." + k: v for k, v in self.right.names.items()}}
+        """The two mixers' tensors under "left.<name>" and "right.<name>", their norms' under "left_norm" and "right_norm"."""
+        own = dict(zip(("left_norm", "right_norm"), self.norm_names)) if self.norm_names else {}
+        return {**{"left." + k: v for k, v in self.left.names.items()}, **{"right." + k: v for k, v in self.right.names.items()}, **own}
+
+
+@dataclass(frozen=True)
+class MambaSpec:
+    """Mamba's selective scan.  W_in h = [x: inner | z: inner]; x passes a causal convolution over time per channel
+    (`conv_taps` taps, the last the current token's, with a bias) and silu; W_x x = [dt: dt_rank | B: state | C: state],
+    dt = softplus(W_dt dt + b) per channel; S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n with A = -exp(A_log),
+    y_c = sum_n S[c, n] C_n + D_c x_c; W_o (y silu(z)).  State per sequence: S [inner, state] in 32-bit and the
+    convolution's last conv_taps - 1 inputs."""
+    width: int
+    inner: int
+    state: int
+    dt_rank: int
+    conv_taps: int
+    kind: str = "mamba"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
+class RgLruSpec:
+    """Griffin's recurrent block: y = gelu_tanh(W_y h + b), u = conv(W_x h + b) (a causal convolution over time per channel,
+    with a bias, no activation), both of `inner`; u falls into `blocks` equal parts, each with square matrices for
+    r = sigmoid(.) and i = sigmoid(.) (biases); log a = -8 r softplus(lam); S <- a S + sqrt(1 - a^2) i u; W_o (S y).
+    State per sequence: S [inner] in 32-bit and the convolution's last conv_taps - 1 inputs."""
+    width: int
+    inner: int
+    blocks: int
+    conv_taps: int
+    kind: str = "rglru"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
+class Mamba2Spec:
+    """Mamba-2.  inner = n_heads * value_dim, N = state; W_in h = [z: inner | x: inner | B: groups N | C: groups N | dt: heads];
+    x, B and C pass a causal convolution over time per channel (with a bias) and silu; dt = softplus(dt + dt_bias); per head
+    (group head // (heads / groups)): S <- exp(-exp(A_log) dt) S + dt B x^T, y = S^T C + D x; the heads' y times silu(z),
+    divided by the root mean square of each of `norm_parts` equal parts (`eps` inside the root), times a weight; W_o.
+    State per sequence: S [heads, value_dim, state] in 32-bit and the convolution's last conv_taps - 1 inputs."""
+    width: int
+    n_heads: int
+    value_dim: int
+    state: int
+    groups: int
+    conv_taps: int
+    norm_parts: int
+    eps: float
+    kind: str = "mamba2"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+    @property
+    def inner(self) -> int:
+        return self.n_heads * self.value_dim
 
 
 @dataclass(frozen=True)
@@ -351,7 +418,9 @@ class RoutedExpertsSpec:
     sigmoid(w_sg . h).
     Options: `scores` "softmax": s = softmax(z) over all experts; `group_score` "max": a group's score is its largest
     choice score; `correction` False: no correction tensor; `shared_gate` False: the shared expert is added as it is.
-    `gated`: every expert (the shared one too) is W_down y with g = min(W_gate h, limit), u = clamp(W_up h, -limit,
+    `normalize`: the weights are the chosen experts' s divided by their sum + `normalize_eps`, times `route_scale`.
+    `gated` "act": an expert is W_down (activation(W_gate h) * (W_up h)) (no shared expert then).
+    `gated` True: every expert (the shared one too) is W_down y with g = min(W_gate h, limit), u = clamp(W_up h, -limit,
     limit), y = g sigmoid(`glu_alpha` g) (u + `glu_shift`) (tensors "gate<e>", "shared_gate_proj"); `limit` for the
     routed experts, `shared_limit` for the shared one (0: no clamp)."""
     width: int
@@ -369,11 +438,13 @@ class RoutedExpertsSpec:
     group_score: str = "top2"
     correction: bool = True
     shared_gate: bool = True
-    gated: bool = False
+    gated: object = False               # False, True (the clamped unit) or "act"
     limit: float = 0.0
     shared_limit: float = 0.0
     glu_alpha: float = 1.702
     glu_shift: float = 1.0
+    normalize: bool = False
+    normalize_eps: float = 0.0
 
 
 @dataclass(frozen=True)
@@ -391,6 +462,8 @@ class BlockSpec:
                                         (norms: "input", "post_input", and with a feed-forward "post_mixer", "post_ffn")
     arrangement "post_norm": the sublayers read the 32-bit stream itself and a norm meets their results only:
         x += norm_1(mixer(x)); x += norm_2(ffn(x))      (norms: "post_input", and with a feed-forward "post_ffn")
+    arrangement "twin_norm": both sublayers read the same x through a norm each, x in 32-bit:
+        x += mixer(norm_1(x)) + ffn(norm_2(x))          (norms: "input", and with a feed-forward "ffn_input")
     arrangement "hyper": the stream in several copies, in 32-bit; each sublayer reads and writes it as its
         `HyperConnectionSpec` says (`connections`: "mixer", and with a feed-forward "ffn"); norms "input", "post_mixer".
     """
@@ -407,9 +480,21 @@ class LayerRun:
     """One entry of the schedule: run layer `layer` against cache entry `cache`.
     A layer may appear in several runs; two runs may name the same cache entry
     when the later one only reads it.  For a layer with several parts that use the
-    cache, `cache` is a tuple with one entry id per such part."""
+    cache, `cache` is a tuple with one entry id per such part.  `enter` = (number of a joint in
+    `ModelSpec.joints`, pass): the joint's step comes right before this run."""
     layer: int
     cache: object
+    enter: Optional[Tuple[int, int]] = None
+
+
+@dataclass(frozen=True)
+class LoopEntrySpec:
+    """What happens to the stream before each pass of a group of layers that runs `times` times in a row: with the
+    embedding's output x0, x <- W_in [x; x0] + step[t], W_in [width, 2 width], step [times, width], t the pass."""
+    width: int
+    times: int
+    kind: str = "loop_entry"
+    names: Mapping[str, str] = field(default_factory=dict)
 
 
 @dataclass(frozen=True)
@@ -474,6 +559,7 @@ class ModelSpec:
     final_norm: Optional[object]            # None: the head sees the last layer's output as it is
     head: object
     stop_tokens: Tuple[int, ...] = ()
+    joints: Tuple[object, ...] = ()         # steps between layers that `LayerRun.enter` names
     bos_token_id: Optional[int] = None
 
     def n_cache_entries(self) -> int:

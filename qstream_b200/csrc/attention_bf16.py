@@ -19,15 +19,15 @@ def _bind():
         _decode = ops.bind("qs_attention_decode_masked", [
             c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p,
             c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_float,
-            c_void_p, c_longlong, c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+            c_void_p, c_longlong, c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
 
 
 def decode(q, n_heads, n_kv_heads, head_dim, scale, window, tok_slot, tok_pos, page_table, page_tokens,
            k_cache, v_cache, max_context, status, out=None, v_head_dim=None, softcap=0.0, gate=None, chunk=0,
-           keep_first=0, sink=None, maps=1, out_dtype=None) -> torch.Tensor:
+           keep_first=0, sink=None, maps=1, out_dtype=None, head_gate=False) -> torch.Tensor:
     """One query token per row against the paged cache, split over the keys and merged.  `v_head_dim`: the values'
     head size where it differs; `softcap` c > 0 caps the scores as c tanh(s / c); `gate` [T, heads * v_head_dim]:
-    the result is multiplied by sigmoid(gate) in the merge.  `chunk`, `keep_first`, `sink`, `maps`, `out_dtype`
+    the result is multiplied by sigmoid(gate) in the merge (`head_gate`: the gate is [T, heads], one value per head).  `chunk`, `keep_first`, `sink`, `maps`, `out_dtype`
     (torch.float32 for a 32-bit result): as for `ops.attention`."""
     _bind()
     T = q.shape[0]
@@ -42,7 +42,7 @@ def decode(q, n_heads, n_kv_heads, head_dim, scale, window, tok_slot, tok_pos, p
                       T, n_heads, n_kv_heads, head_dim, float(scale), int(window), int(max_context),
                       ops.ptr(scratch), ops.ptr(status), dv, float(softcap or 0.0), ops.ptr(gate),
                       gate.stride(0) if gate is not None else 0, int(chunk), int(keep_first), ops.ptr(sink), int(maps),
-                      int(out.dtype == torch.float32), ops.stream()))
+                      int(out.dtype == torch.float32), int(bool(head_gate)), ops.stream()))
     ops.count_launches(1)                                   # split kernel + merge kernel
     return out
 
@@ -67,7 +67,7 @@ def prefill_tiles(batch, device) -> torch.Tensor:
 
 def prefill(q, n_heads, n_kv_heads, head_dim, scale, window, tiles, page_table, page_tokens, k_cache, v_cache,
             status, padded=False, out=None, v_head_dim=None, softcap=0.0, gate=None, chunk=0, keep_first=0, sink=None,
-            maps=1, out_dtype=None) -> torch.Tensor:
+            maps=1, out_dtype=None, head_gate=False) -> torch.Tensor:
     """Many query rows per sequence against the paged cache on the tensor cores (tcgen05).  `v_head_dim`,
     `softcap`, `gate` and the rest: as for `decode`."""
     global _prefill
@@ -75,7 +75,7 @@ def prefill(q, n_heads, n_kv_heads, head_dim, scale, window, tiles, page_table, 
         _prefill = ops.bind("qs_attention_prefill_masked", [
             c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
             c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_float, c_void_p, c_longlong,
-            c_int, c_int, c_void_p, c_int, c_int, c_void_p])
+            c_int, c_int, c_void_p, c_int, c_int, c_int, c_void_p])
     T = q.shape[0]
     dv = int(v_head_dim or head_dim)
     # rows that belong to no sequence (padding) are covered by no tile: give them a defined value
@@ -87,7 +87,8 @@ def prefill(q, n_heads, n_kv_heads, head_dim, scale, window, tiles, page_table, 
                        k_cache.shape[0], ops.ptr(page_table), page_table.shape[1], page_tokens, ops.ptr(tiles),
                        tiles.shape[0], n_heads, n_kv_heads, head_dim, float(scale), int(window), ops.ptr(status),
                        dv, float(softcap or 0.0), ops.ptr(gate), gate.stride(0) if gate is not None else 0,
-                       int(chunk), int(keep_first), ops.ptr(sink), int(maps), int(out.dtype == torch.float32), ops.stream()))
+                       int(chunk), int(keep_first), ops.ptr(sink), int(maps), int(out.dtype == torch.float32), int(bool(head_gate)),
+                       ops.stream()))
     return out
 
 
@@ -100,8 +101,11 @@ def attend(q, spec, step, view, out=None, gate=None, sink=None, out_dtype=None):
     maps = int(getattr(spec, "maps", 1) or 1)
     window = spec.window
     extra = dict(v_head_dim=dv, softcap=spec.softcap, gate=gate, chunk=int(getattr(spec, "chunk", 0) or 0),
-                 keep_first=int(getattr(spec, "keep_first", 0) or 0) if window else 0, sink=sink, maps=maps, out_dtype=out_dtype)
-    if gate is not None and (gate.stride(0) % 8 or gate.data_ptr() % 16 or gate.dtype != torch.bfloat16 or out_dtype == torch.float32):
+                 keep_first=int(getattr(spec, "keep_first", 0) or 0) if window else 0, sink=sink, maps=maps, out_dtype=out_dtype,
+                 head_gate=getattr(spec, "gate", False) == "head")
+    if gate is not None and (gate.dtype != torch.bfloat16 or out_dtype == torch.float32):
+        return None
+    if gate is not None and not extra["head_gate"] and (gate.stride(0) % 8 or gate.data_ptr() % 16):
         return None
     if out is not None and out.dtype != (torch.float32 if out_dtype == torch.float32 else torch.bfloat16):
         return None

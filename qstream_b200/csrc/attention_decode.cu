@@ -412,9 +412,9 @@ __global__ void decode_merge_kernel(__nv_bfloat16* __restrict__ out, size_t ldo,
                                     const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos,
                                     int n_heads, int dh, int window, int max_splits,
                                     const __nv_bfloat16* __restrict__ gate, size_t ldg, int chunk_len, int keep_first,
-                                    const float* __restrict__ sink, int out_f32) {
+                                    const float* __restrict__ sink, int out_f32, int head_gate) {
     // chunk_len, keep_first: as in the split kernel.  sink (may be null): exp(sink[head]) joins the softmax's sum.
-    // out_f32: `out` holds 32-bit floats (ldo counts floats).
+    // out_f32: `out` holds 32-bit floats (ldo counts floats).  head_gate: the gate has one column per head.
     grid_dep_launch();
     const int head = blockIdx.x, t = blockIdx.y;
     __nv_bfloat16* o = out + (size_t)t * ldo + (size_t)head * dh;
@@ -463,7 +463,7 @@ __global__ void decode_merge_kernel(__nv_bfloat16* __restrict__ out, size_t ldo,
                 if (i0 + u < n && s_w[i0 + u] != 0.f) acc += v[u] * s_w[i0 + u];
         }
         float r = acc * inv;
-        if (gate) r *= sigmoid_f32(__bfloat162float(gate[(size_t)t * ldg + (size_t)head * dh + d]));
+        if (gate) r *= sigmoid_f32(__bfloat162float(gate[(size_t)t * ldg + (head_gate ? (size_t)head : (size_t)head * dh + d)]));
         if (out_f32) o32[d] = r; else o[d] = __float2bfloat16_rn(r);
     }
 }
@@ -489,14 +489,15 @@ QS_API long long qs_attention_decode_scratch(int T_tokens, int n_heads, int dh, 
 // The masked form adds: `chunk` c > 0 (without a window): the query sees the keys of its own chunk of c positions counted
 // from 0; `keep_first` n (with a window): the sequence's first n keys stay visible; `sink` (float32 [n_heads], may be
 // null): exp(sink_h) joins each softmax's sum without key or value; `maps` m > 1: K is [n_pages][n_kv_heads][64][m * dh]
-// and n_heads counts m query heads per head, query head j reading key j % m; `out_f32`: out is float32 (ldo in floats).
+// and n_heads counts m query heads per head, query head j reading key j % m; `out_f32`: out is float32 (ldo in floats);
+// `head_gate`: the gate is [T, n_heads], one value per head.
 QS_API int qs_attention_decode_masked(void* out, long long ldo, const void* q, long long ldq, const void* k_cache,
                                       const void* v_cache, const int32_t* page_table, int max_pages, int page_tokens,
                                       const int32_t* tok_slot, const int32_t* tok_pos, int T_tokens, int n_heads,
                                       int n_kv_heads, int dh, float scale, int window, int max_context,
                                       float* scratch, int32_t* status, int dv, float softcap, const void* gate,
                                       long long ldg, int chunk, int keep_first, const float* sink, int maps, int out_f32,
-                                      cudaStream_t stream) {
+                                      int head_gate, cudaStream_t stream) {
     if (T_tokens == 0) return QS_OK;
     if (maps < 1) maps = 1;
     if (window <= 0) keep_first = 0;
@@ -574,7 +575,7 @@ QS_API int qs_attention_decode_masked(void* out, long long ldo, const void* q, l
     if (rc != QS_OK) return rc;
     decode_merge_kernel<<<dim3(n_heads, T_tokens), dv >= 128 ? 128 : 64, (size_t)3 * max_splits * sizeof(float), stream>>>(
         (__nv_bfloat16*)out, (size_t)ldo, scratch, tok_slot, tok_pos, n_heads, dv, window, max_splits,
-        (const __nv_bfloat16*)gate, (size_t)ldg, chunk, keep_first, sink, out_f32);
+        (const __nv_bfloat16*)gate, (size_t)ldg, chunk, keep_first, sink, out_f32, head_gate);
     return qs_check_launch("attention_decode merge");
 }
 
@@ -586,7 +587,7 @@ QS_API int qs_attention_decode_ex(void* out, long long ldo, const void* q, long 
                                   long long ldg, cudaStream_t stream) {
     return qs_attention_decode_masked(out, ldo, q, ldq, k_cache, v_cache, page_table, max_pages, page_tokens, tok_slot, tok_pos,
                                       T_tokens, n_heads, n_kv_heads, dh, scale, window, max_context, scratch, status, dv, softcap,
-                                      gate, ldg, 0, 0, nullptr, 1, 0, stream);
+                                      gate, ldg, 0, 0, nullptr, 1, 0, 0, stream);
 }
 
 QS_API int qs_attention_decode(void* out, long long ldo, const void* q, long long ldq, const void* k_cache,

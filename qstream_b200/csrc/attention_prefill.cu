@@ -39,7 +39,7 @@ constexpr int THREADS = 320;      // producer warp, MMA warp, eight softmax warp
 constexpr float RESCALE_THRESHOLD = 8.0f;        // log2 units
 
 struct TileInfo { int row_start, n_rows, qpos0, slot; };
-struct MaskOpts { int chunk, keep_first, maps, out_f32; const float* sink; };
+struct MaskOpts { int chunk, keep_first, maps, out_f32, head_gate; const float* sink; };
 
 // 2^x on the special-function unit (relative error about 2^-22; -inf gives 0).
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -75,7 +75,7 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
     // mask.keep_first n > 0 (with a window): the sequence's first n keys stay visible; their blocks are walked first.
     // mask.sink (may be null): exp(sink[head]) joins the row's sum, without a key or a value.  mask.maps m > 1: a key
     // row holds m keys of dh side by side and query head j reads key j % m of key head (j / m) / (heads per key head).
-    // mask.out_f32: `out` holds 32-bit floats (ldo counts floats).
+    // mask.out_f32: `out` holds 32-bit floats (ldo counts floats).  mask.head_gate: the gate has one column per head.
     // dh: head size of queries and keys, dv: of values and of the output (NKC covers the larger).  cap_log2 > 0:
     // scores are capped, s <- c tanh(s scale / c), computed as cap_log2 (1 - 2 / (2^(s cap_k2) + 1)) in log2 units
     // with cap_log2 = c log2(e) and cap_k2 = 2 log2(e) scale / c.  gate (may be null): the output row is multiplied
@@ -365,10 +365,11 @@ attention_prefill_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         if (mask.sink && m != -INFINITY) l_all += exp2f(mask.sink[head] * 1.4426950408889634f - m);
         if (ok && !*aborted) {
             tc_fence_after_sync();
-            const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
+            float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
+            if (gate && mask.head_gate && valid) inv *= sigmoid_f32(__bfloat162float(gate[(size_t)(tile.row_start + r) * ldg + head]));
             __nv_bfloat16* orow = out + (size_t)(tile.row_start + r) * ldo + (size_t)head * dv;
             float* orow32 = reinterpret_cast<float*>(out) + (size_t)(tile.row_start + r) * ldo + (size_t)head * dv;
-            const __nv_bfloat16* grow = gate ? gate + (size_t)(tile.row_start + r) * ldg + (size_t)head * dv : nullptr;
+            const __nv_bfloat16* grow = gate && !mask.head_gate ? gate + (size_t)(tile.row_start + r) * ldg + (size_t)head * dv : nullptr;
             for (int c = half; c * 32 < dv; c += 2) {
                 uint32_t o[32];
                 tmem_load_32x32(tmem_base + lane_base + O_COL + (uint32_t)(c * 32), o);
@@ -485,14 +486,14 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 // from 0; `keep_first` n (with a window): the sequence's first n keys stay visible; `sink` (float32 [n_heads], may be
 // null): exp(sink_h) joins each softmax's sum without key or value; `maps` m > 1: K is [n_pages][n_kv_heads][64][m * dh]
 // and n_heads counts m query heads per head, query head j reading key j % m; `out_f32`: out is float32 (ldo in floats,
-// rows 16-byte aligned), which excludes a gate.
+// rows 16-byte aligned), which excludes a gate; `head_gate`: the gate is [T, n_heads], one value per head (any row stride).
 QS_API int qs_attention_prefill_masked(void* out, long long ldo, const void* q, long long ldq, int T_tokens,
                                        const void* k_cache, const void* v_cache, int n_pages,
                                        const int32_t* page_table, int max_pages, int page_tokens,
                                        const int32_t* tiles, int n_tiles, int n_heads, int n_kv_heads, int dh,
                                        float scale, int window, int32_t* status, int dv, float softcap, const void* gate,
                                        long long ldg, int chunk, int keep_first, const float* sink, int maps, int out_f32,
-                                       cudaStream_t stream) {
+                                       int head_gate, cudaStream_t stream) {
     if (n_tiles == 0 || T_tokens == 0) return QS_OK;
     if (maps < 1) maps = 1;
     QS_REQUIRE(chunk >= 0 && keep_first >= 0 && !(chunk > 0 && window > 0), "attention_prefill: a window of %d and chunks of %d", window, chunk);
@@ -500,7 +501,7 @@ QS_API int qs_attention_prefill_masked(void* out, long long ldo, const void* q, 
                n_heads, maps, n_kv_heads);
     QS_REQUIRE(!out_f32 || (!gate && ldo % 4 == 0), "attention_prefill: 32-bit results take no gate and rows of whole 16 bytes");
     QS_REQUIRE(dv % 16 == 0 && dv >= 16 && dv <= 256, "attention_prefill: value head size %d must be a multiple of 16 up to 256", dv);
-    QS_REQUIRE(!gate || (ldg % 8 == 0 && ((uintptr_t)gate % 16) == 0), "attention_prefill: the gate's rows must be 16-byte aligned");
+    QS_REQUIRE(!gate || head_gate || (ldg % 8 == 0 && ((uintptr_t)gate % 16) == 0), "attention_prefill: the gate's rows must be 16-byte aligned");
     QS_REQUIRE(scale > 0.f && softcap >= 0.f, "attention_prefill: the scale must be positive and the cap not negative");
     QS_REQUIRE(T_tokens > 0 && n_tiles > 0 && n_heads > 0 && n_kv_heads > 0 && n_pages > 0, "attention_prefill: bad sizes");
     QS_REQUIRE(page_tokens == BN, "attention_prefill: pages of %d tokens, the kernel is built for %d", page_tokens, BN);
@@ -520,7 +521,7 @@ QS_API int qs_attention_prefill_masked(void* out, long long ldo, const void* q, 
     const float cap_log2 = softcap > 0.f ? softcap * log2e : 0.f;
     const float cap_k2 = softcap > 0.f ? 2.0f * log2e * scale / softcap : 0.f;
     const TileInfo* ti = reinterpret_cast<const TileInfo*>(tiles);
-    const MaskOpts mask = {chunk, keep_first, maps, out_f32, sink};
+    const MaskOpts mask = {chunk, keep_first, maps, out_f32, head_gate, sink};
     const int nkc = ((dh > dv ? dh : dv) + KC - 1) / KC;
 #define GO(NKC) return launch<NKC>(mq, mk, mv, out, ldo, ti, n_tiles, page_table, max_pages, n_heads, n_kv_heads, dh, \
                                    scale_log2, window, status, dv, cap_log2, cap_k2, gate, ldg, mask, stream)
@@ -539,7 +540,7 @@ QS_API int qs_attention_prefill_ex(void* out, long long ldo, const void* q, long
                                    long long ldg, cudaStream_t stream) {
     return qs_attention_prefill_masked(out, ldo, q, ldq, T_tokens, k_cache, v_cache, n_pages, page_table, max_pages, page_tokens,
                                        tiles, n_tiles, n_heads, n_kv_heads, dh, scale, window, status, dv, softcap, gate, ldg,
-                                       0, 0, nullptr, 1, 0, stream);
+                                       0, 0, nullptr, 1, 0, 0, stream);
 }
 
 QS_API int qs_attention_prefill(void* out, long long ldo, const void* q, long long ldq, int T_tokens,

@@ -141,6 +141,8 @@ __device__ __forceinline__ float gelu_erf(float v) {
 // sigmoid(v) = 1 / (1 + exp(-v)) and silu(v) = v sigmoid(v), in 32-bit with the full-precision exponential.
 __device__ __forceinline__ float sigmoid_f32(float v) { return 1.0f / (1.0f + expf(-v)); }
 __device__ __forceinline__ float silu_f32(float v) { return v / (1.0f + expf(-v)); }
+// log(1 + exp(v)) without overflow.
+__device__ __forceinline__ float softplus_f32(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 __device__ __forceinline__ float apply_activation(float v, int act) {
     if (act == QS_ACT_GELU_TANH) return gelu_tanh(v);

@@ -17,8 +17,6 @@ namespace {
 
 constexpr int MAX_TAPS = 8;
 
-__device__ __forceinline__ float softplus_f32(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
-
 template <typename TI>
 __global__ void delta_prepare_kernel(float* __restrict__ qo, float* __restrict__ ko, float* __restrict__ vo,
                                      float* __restrict__ go, float* __restrict__ bo,

@@ -111,8 +111,8 @@ __global__ void latent_q_rotate_kernel(T* __restrict__ q_abs, size_t ldqa, const
 // fixed order.
 constexpr int HL_T = 8, HL_N = 32;
 
-template <typename T>
-__global__ void head_linear_kernel(T* __restrict__ out, size_t ldo, size_t head_o, const T* __restrict__ x, size_t ldx,
+template <typename T, typename TO>
+__global__ void head_linear_kernel(TO* __restrict__ out, size_t ldo, size_t head_o, const T* __restrict__ x, size_t ldx,
                                    size_t head_x, const T* __restrict__ w, int n_tokens, int N, int K) {
     extern __shared__ float xs[];                       // [HL_T][K]
     grid_dep_launch();
@@ -139,7 +139,7 @@ __global__ void head_linear_kernel(T* __restrict__ out, size_t ldo, size_t head_
 #pragma unroll
         for (int tt = 0; tt < HL_T; ++tt) {
             const float total = warp_sum(acc[tt]);
-            if (tt < nt && lane == 0) out[(size_t)(t0 + tt) * ldo + (size_t)h * head_o + n] = from_f32<T>(total);
+            if (tt < nt && lane == 0) out[(size_t)(t0 + tt) * ldo + (size_t)h * head_o + n] = from_f32<TO>(total);
         }
     }
 }
@@ -197,20 +197,21 @@ QS_API int qs_latent_q_rotate(void* q_abs, long long ldqa, const void* q, long l
 }
 
 // x: head h's K inputs of token t at x[t * ldx + h * head_x + k]; w [H][N][K] contiguous; out likewise with ldo, head_o.
-QS_API int qs_head_linear(void* out, long long ldo, long long head_o, const void* x, long long ldx, long long head_x,
-                          const void* w, int dtype, int T_tokens, int H, int N, int K, cudaStream_t stream) {
+QS_API int qs_head_linear(void* out, int out_dtype, long long ldo, long long head_o, const void* x, long long ldx,
+                          long long head_x, const void* w, int dtype, int T_tokens, int H, int N, int K, cudaStream_t stream) {
     if (T_tokens == 0) return QS_OK;
     QS_REQUIRE(T_tokens > 0 && H > 0 && N > 0 && K > 0 && H <= 65535, "head_linear: bad sizes");
     const size_t smem = (size_t)HL_T * K * sizeof(float);
     QS_REQUIRE(smem <= 200 * 1024, "head_linear: %d inputs per head do not fit shared memory", K);
     dim3 grid(H, (N + HL_N - 1) / HL_N, (T_tokens + HL_T - 1) / HL_T);
     cudaError_t e = cudaSuccess;
-#define GO(T) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(head_linear_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-    if (e == cudaSuccess) e = qs_launch_dependent(head_linear_kernel<T>, grid, dim3(256), smem, stream, (T*)out, (size_t)ldo, (size_t)head_o, \
+#define GO(T, TO) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(head_linear_kernel<T, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+    if (e == cudaSuccess) e = qs_launch_dependent(head_linear_kernel<T, TO>, grid, dim3(256), smem, stream, (TO*)out, (size_t)ldo, (size_t)head_o, \
         (const T*)x, (size_t)ldx, (size_t)head_x, (const T*)w, T_tokens, N, K); } while (0)
-    if (dtype == QS_F32) GO(float);
-    else if (dtype == QS_BF16) GO(__nv_bfloat16);
-    else return qs_fail(QS_ERR_INVALID_INPUT, "head_linear: unknown dtype %d", dtype);
+    if (dtype == QS_F32 && out_dtype == QS_F32) GO(float, float);
+    else if (dtype == QS_BF16 && out_dtype == QS_BF16) GO(__nv_bfloat16, __nv_bfloat16);
+    else if (dtype == QS_BF16 && out_dtype == QS_F32) GO(__nv_bfloat16, float);
+    else return qs_fail(QS_ERR_INVALID_INPUT, "head_linear: unsupported types in=%d out=%d", dtype, out_dtype);
 #undef GO
     if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "head_linear: %s", cudaGetErrorString(e));
     return qs_check_launch("head_linear");

@@ -5,7 +5,8 @@
 //                 stay (the others count as minus infinity); the `top` largest choice scores win (equal scores: the
 //                 lower index); weights s * scale of the winners, not renormalised; optionally sigmoid of one more
 //                 logit per token (the gate of a shared expert).  `score_kind` 1: s = softmax(z) over all experts
-//                 instead of the sigmoid; `group_kind` 1: a group's score is its largest choice score
+//                 instead of the sigmoid; `group_kind` 1: a group's score is its largest choice score; `renorm_eps` >= 0:
+//                 the winners' scores are divided by their sum + renorm_eps
 //   few tokens    moe_expert_up / moe_expert_down: every (token, chosen expert) pair reads its expert's matrices
 //                 through the routing table on the device, so a step can be captured and replayed
 //   many tokens   moe_sort orders the pairs by expert; the caller runs one matrix product per expert over its rows
@@ -22,7 +23,7 @@ constexpr int MAX_EXPERTS = 1024;
 __global__ void moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ wts, float* __restrict__ shared_gate,
                                  const float* __restrict__ z, size_t ldz, const void* __restrict__ corr, int corr_dtype,
                                  int T, int E, int top, int groups, int keep, float scale, int gate_col, int score_kind,
-                                 int group_kind) {
+                                 int group_kind, float renorm_eps) {
     extern __shared__ float sm[];                       // per warp: s [E], choice [E], group score [groups]
     grid_dep_launch();
     grid_dep_wait();
@@ -80,6 +81,12 @@ __global__ void moe_route_kernel(int32_t* __restrict__ idx, float* __restrict__ 
             wts[(size_t)t * top + j] = s[best] * scale;
             choice[best] = -INFINITY;
         }
+        if (renorm_eps >= 0.f) {                            // the chosen scores made to sum to one, in the order of choice
+            float sum = 0.f;
+            for (int j = 0; j < top; ++j) sum += s[idx[(size_t)t * top + j]];
+            const float inv = scale / (sum + renorm_eps);
+            for (int j = 0; j < top; ++j) wts[(size_t)t * top + j] = s[idx[(size_t)t * top + j]] * inv;
+        }
     }
 }
 
@@ -103,12 +110,13 @@ __device__ __forceinline__ float warp_dot(const T* __restrict__ w, const float* 
 }
 
 // hidden[pair, f] = act(W_up[e][f, :] . h[token, :]) for pair = token * top + j, e = idx[pair]: a block stages the
-// token's row in shared memory as 32-bit floats, a warp takes one hidden unit at a time.
+// token's row in shared memory as 32-bit floats, a warp takes one hidden unit at a time.  `gated`: an expert's matrix holds
+// F gate rows above its F up rows, and hidden = act(gate . h) * (up . h).
 template <typename T>
 __global__ void moe_expert_up_kernel(T* __restrict__ hidden, size_t ldh, const T* __restrict__ x, size_t ldx,
                                      const T* __restrict__ w_up, const int32_t* __restrict__ idx,
                                      const int32_t* __restrict__ tok_slot, int top, int D, int F, int rows_per_block, int act,
-                                     int vec) {
+                                     int vec, int gated) {
     extern __shared__ __align__(16) float xs[];
     grid_dep_launch();
     grid_dep_wait();
@@ -121,10 +129,11 @@ __global__ void moe_expert_up_kernel(T* __restrict__ hidden, size_t ldh, const T
     }
     for (int i = threadIdx.x; i < D; i += blockDim.x) xs[i] = to_f32(x[(size_t)t * ldx + i]);
     __syncthreads();
-    const T* w = w_up + (size_t)idx[pair] * F * D;
+    const T* w = w_up + (size_t)idx[pair] * (gated ? 2 : 1) * F * D;
     for (int f = f0 + warp; f < min(F, f0 + rows_per_block); f += warps) {
         const float acc = warp_dot(w + (size_t)f * D, xs, D, lane, vec != 0);
-        if (lane == 0) hidden[(size_t)pair * ldh + f] = from_f32<T>(apply_activation_wide(acc, act));
+        const float mul = gated ? warp_dot(w + (size_t)(F + f) * D, xs, D, lane, vec != 0) : 1.0f;
+        if (lane == 0) hidden[(size_t)pair * ldh + f] = from_f32<T>(apply_activation_wide(acc, act) * mul);
     }
 }
 
@@ -215,7 +224,7 @@ __global__ void moe_combine_kernel(float* __restrict__ out, size_t ldo, const TY
 
 QS_API int qs_moe_route(int32_t* idx, float* wts, float* shared_gate, const float* z, long long ldz, const void* corr,
                         int corr_dtype, int T, int E, int top, int groups, int keep, float scale, int gate_col,
-                        int score_kind, int group_kind, cudaStream_t stream) {
+                        int score_kind, int group_kind, float renorm_eps, cudaStream_t stream) {
     if (T == 0) return QS_OK;
     QS_REQUIRE(T > 0 && E > 0 && E <= MAX_EXPERTS && top > 0 && top <= E, "moe_route: bad sizes T=%d E=%d top=%d", T, E, top);
     QS_REQUIRE(groups > 0 && E % groups == 0 && keep > 0 && keep <= groups, "moe_route: %d experts in %d groups, %d kept", E, groups, keep);
@@ -224,14 +233,14 @@ QS_API int qs_moe_route(int32_t* idx, float* wts, float* shared_gate, const floa
     const size_t smem = (size_t)warps * (2 * E + groups) * sizeof(float);
     cudaError_t e = qs_launch_dependent(moe_route_kernel, dim3((T + warps - 1) / warps), dim3(warps * 32), smem, stream, idx, wts,
                                         shared_gate, z, (size_t)ldz, corr, corr_dtype, T, E, top, groups, keep, scale, gate_col, score_kind,
-                                        group_kind);
+                                        group_kind, renorm_eps);
     if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "moe_route: %s", cudaGetErrorString(e));
     return qs_check_launch("moe_route");
 }
 
 QS_API int qs_moe_expert_up(void* hidden, long long ldh, const void* x, long long ldx, const void* w_up, int dtype,
                             const int32_t* idx, const int32_t* tok_slot, int T, int top, int D, int F, int act,
-                            cudaStream_t stream) {
+                            int gated, cudaStream_t stream) {
     if (T == 0) return QS_OK;
     QS_REQUIRE(T > 0 && top > 0 && D > 0 && F > 0, "moe_expert_up: bad sizes");
     QS_REQUIRE((size_t)D * sizeof(float) <= 200 * 1024, "moe_expert_up: width %d does not fit shared memory", D);
@@ -242,7 +251,7 @@ QS_API int qs_moe_expert_up(void* hidden, long long ldh, const void* x, long lon
     cudaError_t e = cudaSuccess;
 #define GO(TT) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_expert_up_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e == cudaSuccess) e = qs_launch_dependent(moe_expert_up_kernel<TT>, grid, dim3(256), smem, stream, (TT*)hidden, (size_t)ldh, (const TT*)x, \
-        (size_t)ldx, (const TT*)w_up, idx, tok_slot, top, D, F, rows_per_block, act, vec); } while (0)
+        (size_t)ldx, (const TT*)w_up, idx, tok_slot, top, D, F, rows_per_block, act, vec, gated); } while (0)
     if (dtype == QS_F32) GO(float);
     else if (dtype == QS_BF16) GO(__nv_bfloat16);
     else return qs_fail(QS_ERR_INVALID_INPUT, "moe_expert_up: unknown dtype %d", dtype);

@@ -74,17 +74,31 @@ _SIGNATURES = {
                          c_void_p, c_int, c_longlong, c_int, c_int, c_int, c_float, c_void_p], c_int),
     "qs_branch_norm": ([c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_int, c_longlong, c_void_p,
                         c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p], c_int),
+    "qs_stream_tanh_norm": ([c_void_p, c_longlong, c_int, c_int, c_float, *([c_void_p, c_longlong, c_float, c_void_p, c_int] * 3), c_int,
+                             *([c_void_p, c_longlong, c_float, c_void_p, c_int, c_void_p, c_int] * 2), c_void_p], c_int),
+    "qs_short_conv": ([c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_longlong,
+                       c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p], c_int),
+    "qs_conv_keep": ([c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], c_int),
+    "qs_selective_scan": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_longlong, c_void_p,
+                           c_longlong, c_void_p, c_void_p, c_longlong, c_int, c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int,
+                           c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p], c_int),
+    "qs_gated_lru": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_void_p, c_void_p, c_longlong, c_int,
+                      c_void_p, c_longlong, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                      c_void_p, c_void_p], c_int),
+    "qs_ssd_gates": ([c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p], c_int),
+    "qs_ssd_output": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p,
+                       c_int, c_int, c_int, c_int, c_int, c_float, c_void_p], c_int),
     "qs_latent_prepare": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_int, c_void_p, c_longlong,
                            c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_float, c_float, c_int, c_void_p, c_void_p,
                            c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p], c_int),
     "qs_latent_q_rotate": ([c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p], c_int),
-    "qs_head_linear": ([c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int,
+    "qs_head_linear": ([c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_longlong, c_longlong, c_void_p, c_int, c_int, c_int,
                         c_int, c_int, c_void_p], c_int),
     "qs_moe_route": ([c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
-                      c_int, c_float, c_int, c_int, c_int, c_void_p], c_int),
+                      c_int, c_float, c_int, c_int, c_int, c_float, c_void_p], c_int),
     "qs_moe_expert_up": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                          c_int, c_int, c_int, c_void_p], c_int),
+                          c_int, c_int, c_int, c_int, c_void_p], c_int),
     "qs_moe_expert_down": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
                             c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p], c_int),
     "qs_moe_sort": ([c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p], c_int),
@@ -522,6 +536,8 @@ def state_scan(mode: str, q, k, v, state, seq_start, seq_slot, n_seq, n_heads, k
     given each its starting state, the chunk's outputs).  In mode "decay" `q_scale` multiplies q as well.
     mode "gla": S <- diag(w_t) S + k v^T, o = S^T (q q_scale), w_t = sigmoid(decay_logits)^`decay_power` per token and key
     channel (float32 [T, heads * key_dim]), taken in 32-bit inside the walk.
+    mode "ssd": S <- a_t S + b_t k v^T, o = S^T (q q_scale) with a = `token_decay`, b = `token_weight` (float32 [T, heads]);
+    q and k hold heads / `qk_group` heads, as in mode "delta".
     `chunks` = (chunk_start, chunk_ids, seq_chunk, n_chunks), int32 device tensors: every sequence of the step cut
     into consecutive chunks (rows chunk_start[c] .. chunk_start[c + 1] of the packed batch; sequence s owns chunks
     seq_chunk[s] .. seq_chunk[s + 1]; chunk_ids = 0 .. n_chunks - 1).  The chunks then run side by side and a
@@ -547,10 +563,10 @@ def state_scan(mode: str, q, k, v, state, seq_start, seq_slot, n_seq, n_heads, k
         decay_logits = key_decay
         if key_decay.dtype != torch.float32 or token_weight.dtype != torch.float32:
             raise QStreamError(QsError.INVALID_INPUT, "state_scan: the delta rule takes float32 decays and step sizes")
-    if mode == "gated" and (token_decay.dtype != torch.float32 or token_decay.stride() != token_weight.stride()):
+    if mode in ("gated", "ssd") and (token_decay.dtype != torch.float32 or token_decay.stride() != token_weight.stride()):
         raise QStreamError(QsError.INVALID_INPUT, "state_scan: the tokens' decays and weights must be float32 of one layout")
     check(library().qs_state_scan(
-        {"decay": 0, "wkv": 1, "gated": 2, "delta": 3, "gla": 4}[mode], ptr(o), o.stride(0) if o is not None else 0, ptr(q), q.stride(0),
+        {"decay": 0, "wkv": 1, "gated": 2, "delta": 3, "gla": 4, "ssd": 5}[mode], ptr(o), o.stride(0) if o is not None else 0, ptr(q), q.stride(0),
         ptr(k), k.stride(0), ptr(v), v.stride(0) if v is not None else 0,
         dtype_code(q), ptr(decay_logits), decay_logits.stride(0) if decay_logits is not None else 0, ptr(head_decay),
         ptr(bonus), _code(bonus), ptr(state), state.stride(0), _int32(seq_start, "seq_start"),
@@ -670,6 +686,135 @@ def branch_norm(x, weight, eps: float, center: bool, out_dtype=None, branch=None
     return h
 
 
+def stream_tanh_norm(x, branches=(), eps: float = 0.0, reads=(), out_dtype=None):
+    """The 32-bit stream x [T, D] written and read in one pass.  `branches`: up to three (factor, y, weight or None), y
+    float32 [T, D]: x <- x + sum of factor * y, a branch with a weight divided by its root mean square over D first
+    (y / sqrt(mean(y^2) + eps) * weight); in place.  `reads`: up to two (alpha, weight, shift, out or None), each giving
+    tanh(alpha x) * weight + shift of the new x, or, with weight None, x itself, in `out_dtype` (or into `out`, a view with
+    contiguous rows of that type).  Returns the list of reads."""
+    rows, D, ldx = _rows(x)
+    if x.dtype != torch.float32 or len(branches) > 3 or len(reads) > 2:
+        raise QStreamError(QsError.INVALID_INPUT, "stream_tanh_norm: a float32 stream, up to three branches and two reads")
+    args = []
+    for mult, y, w in [*branches, *[(0.0, None, None)] * (3 - len(branches))]:
+        ld = 0
+        if y is not None:
+            r2, D2, ld = _rows(y)
+            if (r2, D2) != (rows, D) or y.dtype != torch.float32 or (w is not None and w.numel() != D):
+                raise QStreamError(QsError.INVALID_INPUT, "stream_tanh_norm: a branch differs from the stream in shape or type")
+        args += [ptr(y), ld, float(mult), ptr(w), _code(w)]
+    hs, out_args = [], []
+    dtype = out_dtype or x.dtype
+    for alpha, w, b, out in reads:
+        h = out if out is not None else torch.empty((rows, D), dtype=dtype, device=x.device)
+        if h.shape != (rows, D) or h.stride(1) != 1 or h.dtype != dtype or (w is not None and (w.numel() != D or b.numel() != D)):
+            raise QStreamError(QsError.INVALID_INPUT, "stream_tanh_norm: a read's output or weights do not fit")
+        hs.append(h)
+        out_args += [ptr(h), h.stride(0), float(alpha), ptr(w), _code(w), ptr(b), _code(b)]
+    out_args += [None, 0, 0.0, None, 0, None, 0] * (2 - len(reads))
+    check(library().qs_stream_tanh_norm(ptr(x), ldx, rows, D, float(eps), *args, F32 if dtype == torch.float32 else BF16, *out_args, stream()))
+    return hs
+
+
+# ------------------------------------------------------------------------------- recurrences with a state per channel
+
+def short_conv(x, taps, bias, held, tok_slot, tok_pos, activation=None, decode=False) -> torch.Tensor:
+    """A causal convolution over time per channel: out[t] = act(bias + sum_j taps[:, n - 1 - j] x[t - j]) for x [T, C], taps
+    [C, n]; the n - 1 inputs before a step's first token come from `held` [slots, n - 1, C] (None for one tap).  `decode`:
+    every row is one token of its own sequence, and `held` is brought up to date in the same pass; otherwise call
+    `conv_keep` afterwards."""
+    T, C, ldx = _rows(x)
+    n = taps.shape[1]
+    if taps.shape[0] != C or not taps.is_contiguous() or (bias is not None and bias.numel() != C) or \
+            (n > 1 and (held is None or held.dtype != x.dtype or held.shape[1:] != (n - 1, C))):
+        raise QStreamError(QsError.INVALID_INPUT, "short_conv: operands do not fit")
+    out = torch.empty((T, C), dtype=x.dtype, device=x.device)
+    check(library().qs_short_conv(ptr(out), C, ptr(x), ldx, dtype_code(x), ptr(taps), dtype_code(taps), ptr(bias), _code(bias), n,
+                                  ptr(held), held.stride(0) if held is not None else 0, _int32(tok_slot, "tok_slot"),
+                                  _int32(tok_pos, "tok_pos"), T, C, ACTIVATIONS[activation], int(bool(decode)), stream()))
+    return out
+
+
+def conv_keep(held, x, seq_start, seq_slot, n_seq: int) -> None:
+    """Leave in `held` [slots, n - 1, C] the last n - 1 inputs of what each of the step's sequences held and the step brought."""
+    _, C, ldx = _rows(x)
+    check(library().qs_conv_keep(ptr(held), held.stride(0), ptr(x), ldx, dtype_code(x), C, held.shape[1] + 1,
+                                 _int32(seq_start, "seq_start"), _int32(seq_slot, "seq_slot"), int(n_seq), stream()))
+
+
+def _channel_chunks(chunks, per_chunk: int, channels: int, device):
+    """The chunk arguments of a scan with a state per channel, with their scratch."""
+    if chunks is None:
+        return None, None, 0, None, None, None
+    chunk_start, chunk_ids, seq_chunk, n_chunks = chunks
+    return (chunk_start, chunk_ids, n_chunks, seq_chunk, torch.empty((n_chunks, per_chunk), dtype=torch.float32, device=device),
+            torch.empty((n_chunks, channels), dtype=torch.float32, device=device))
+
+
+def selective_scan(x, raw, a2, B, C, D, z, state, seq_start, seq_slot, n_seq: int, chunks=None) -> torch.Tensor:
+    """Mamba's selective scan: dt = softplus(raw), S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,
+    y_c = sum_n S[c, n] C_n + D_c x_c, returned as y silu(z) [T, inner] in x's type.  raw float32 [T, inner];
+    a2 = A log2(e) float32 [inner, N]; B, C [T, N] views in x's type; D float32 [inner]; `state` float32
+    [slots, inner, N], updated in place.  `chunks`: as for `state_scan`."""
+    T, inner, ldx = _rows(x)
+    N = a2.shape[1]
+    if raw.dtype != torch.float32 or a2.dtype != torch.float32 or D.dtype != torch.float32 or state.dtype != torch.float32 or \
+            B.dtype != x.dtype or C.dtype != x.dtype or z.dtype != x.dtype or a2.shape[0] != inner or B.shape != (T, N) or C.shape != (T, N) \
+            or raw.shape != (T, inner) or z.shape != (T, inner) or not a2.is_contiguous():
+        raise QStreamError(QsError.INVALID_INPUT, "selective_scan: operands do not fit")
+    out = torch.empty((T, inner), dtype=x.dtype, device=x.device)
+    c_start, c_ids, n_chunks, s_chunk, c_state, c_logs = _channel_chunks(chunks, inner * N, inner, x.device)
+    check(library().qs_selective_scan(
+        ptr(out), inner, ptr(x), ldx, ptr(raw), raw.stride(0), ptr(a2), ptr(B), B.stride(0), ptr(C), C.stride(0), ptr(D), ptr(z),
+        z.stride(0), dtype_code(x), ptr(state), state.stride(0), _int32(seq_start, "seq_start"), _int32(seq_slot, "seq_slot"),
+        int(n_seq), T, inner, N, ptr(c_start), ptr(c_ids), int(n_chunks), ptr(s_chunk), ptr(c_state), ptr(c_logs), stream()))
+    if chunks is not None:
+        count_launches(2)
+    return out
+
+
+def gated_lru(u, gates, bias, rate, y, state, block: int, seq_start, seq_slot, n_seq: int, chunks=None) -> torch.Tensor:
+    """The gated linear recurrent unit: per block of `block` channels `gates` float32 [T, 2 n] and `bias` float32 [2 n] hold
+    (r | i) before the sigmoid; log a = -rate sigmoid(r), S <- a S + sqrt(1 - a^2) sigmoid(i) u; returns S gelu_tanh(y) [T, n]
+    in u's type.  rate float32 [n]; `state` float32 [slots, n], updated in place.  `chunks`: as for `state_scan`."""
+    T, n, ldu = _rows(u)
+    if gates.dtype != torch.float32 or bias.dtype != torch.float32 or rate.dtype != torch.float32 or state.dtype != torch.float32 or \
+            gates.shape != (T, 2 * n) or bias.numel() != 2 * n or rate.numel() != n or y.shape != (T, n) or y.dtype != u.dtype or n % block:
+        raise QStreamError(QsError.INVALID_INPUT, "gated_lru: operands do not fit")
+    out = torch.empty((T, n), dtype=u.dtype, device=u.device)
+    c_start, c_ids, n_chunks, s_chunk, c_state, c_logs = _channel_chunks(chunks, n, n, u.device)
+    check(library().qs_gated_lru(
+        ptr(out), n, ptr(u), ldu, ptr(gates), gates.stride(0), ptr(bias), ptr(rate), ptr(y), y.stride(0), dtype_code(u), ptr(state),
+        state.stride(0), _int32(seq_start, "seq_start"), _int32(seq_slot, "seq_slot"), int(n_seq), T, n, int(block), ptr(c_start),
+        ptr(c_ids), int(n_chunks), ptr(s_chunk), ptr(c_state), ptr(c_logs), stream()))
+    if chunks is not None:
+        count_launches(2)
+    return out
+
+
+def ssd_gates(raw, a_log):
+    """dt = softplus(raw) and a = exp(-exp(a_log_h) dt), each float32 [T, heads]; raw float32 [T, heads], bias included."""
+    T, H, ldr = _rows(raw)
+    if raw.dtype != torch.float32 or a_log.dtype != torch.float32 or a_log.numel() != H:
+        raise QStreamError(QsError.INVALID_INPUT, "ssd_gates: float32 step sizes and rates, one per head")
+    both = torch.empty((2, T, H), dtype=torch.float32, device=raw.device)
+    check(library().qs_ssd_gates(ptr(both[0]), ptr(both[1]), ptr(raw), ldr, ptr(a_log), T, H, stream()))
+    return both[0], both[1]
+
+
+def ssd_output(o, x, z, D, weight, value_dim: int, parts: int, eps: float) -> torch.Tensor:
+    """v = (o + D_h x) silu(z) for o float32 [T, n] and x, z [T, n] (heads of `value_dim`; D float32, one per head); each of
+    `parts` equal parts of v divided by its root mean square, times `weight` [n]; in x's type."""
+    T, n, ldo = _rows(o)
+    if o.dtype != torch.float32 or x.shape != (T, n) or z.shape != (T, n) or x.dtype != z.dtype or D.dtype != torch.float32 or \
+            D.numel() * value_dim != n or weight.numel() != n:
+        raise QStreamError(QsError.INVALID_INPUT, "ssd_output: operands do not fit")
+    out = torch.empty((T, n), dtype=x.dtype, device=x.device)
+    check(library().qs_ssd_output(ptr(out), n, ptr(o), ldo, ptr(x), x.stride(0), ptr(z), z.stride(0), dtype_code(x), ptr(D), ptr(weight),
+                                  dtype_code(weight), T, n, int(value_dim), int(parts), float(eps), stream()))
+    return out
+
+
 def latent_prepare(dq, q_norm, q_rank, dkv, kv_norm, kv_rank, rot_dim, rot_dims, freq, mag, eps, tok_slot, tok_pos,
                    page_table, page_tokens, k_cache, v_cache, status, interleaved=False):
     """RMS norm of the query latent dq [T, q_rank] -> returned; RMS norm of the key latent dkv[:, :kv_rank] and the
@@ -702,12 +847,12 @@ def latent_q_rotate(q_abs, q, n_heads, dim, rot_dim, kv_rank, rot_dims, freq, ma
 def head_linear(out, x, w, n_heads: int) -> None:
     """out[:, h * N : (h + 1) * N] = x[:, h * Kx : h * Kx + K] @ w[h].T for every head h, where w is [heads, N, K], out
     is [T, heads * N'] with N' >= N (head h's results at the start of its N' columns) and x is [T, heads * Kx] with
-    Kx >= K: one launch for all heads, for steps of few tokens; 32-bit sums."""
+    Kx >= K: one launch for all heads, for steps of few tokens; 32-bit sums (and, where `out` is float32, results)."""
     H, N, K = w.shape
     T = x.shape[0]
-    if H != n_heads or x.shape[1] % H or out.shape[1] % H or w.dtype != x.dtype or out.dtype != x.dtype or not w.is_contiguous():
+    if H != n_heads or x.shape[1] % H or out.shape[1] % H or w.dtype != x.dtype or out.dtype not in (x.dtype, torch.float32) or not w.is_contiguous():
         raise QStreamError(QsError.INVALID_INPUT, "head_linear: operands do not fit")
-    check(library().qs_head_linear(ptr(out), out.stride(0), out.shape[1] // H, ptr(x), x.stride(0), x.shape[1] // H, ptr(w),
+    check(library().qs_head_linear(ptr(out), dtype_code(out), out.stride(0), out.shape[1] // H, ptr(x), x.stride(0), x.shape[1] // H, ptr(w),
                                    dtype_code(x), T, H, N, K, stream()))
 
 
@@ -717,7 +862,7 @@ def head_products(out, x, w, n_heads: int) -> None:
     from . import gemm_tc
     H, N, K = w.shape
     T = x.shape[0]
-    if H != n_heads or x.shape[1] % H or out.shape[1] % H or w.dtype != x.dtype or out.dtype != x.dtype or not w.is_contiguous():
+    if H != n_heads or x.shape[1] % H or out.shape[1] % H or w.dtype != x.dtype or out.dtype not in (x.dtype, torch.float32) or not w.is_contiguous():
         raise QStreamError(QsError.INVALID_INPUT, "head_products: operands do not fit")
     head_x, head_o = x.shape[1] // H, out.shape[1] // H
     use_tc = gemm_tc.takes(x[:, :K], w[0]) and head_x % 8 == 0
@@ -733,10 +878,11 @@ def head_products(out, x, w, n_heads: int) -> None:
 
 # ------------------------------------------------------------------------------- routed experts
 
-def moe_route(z, correction, n_experts, top, groups, keep, scale, gate_col=-1, scores="sigmoid", group_score="top2"):
+def moe_route(z, correction, n_experts, top, groups, keep, scale, gate_col=-1, scores="sigmoid", group_score="top2", renorm_eps=None):
     """z float32 [T, >= n_experts] router logits.  Returns (idx int32 [T, top], weights float32 [T, top], shared gate
     float32 [T] = sigmoid(z[:, gate_col]) or None): see csrc/moe.cu for the rule.  `scores`: "sigmoid" or "softmax" (over
-    all experts); `group_score`: "top2" (the sum of a group's two largest) or "max"; `correction` may be None."""
+    all experts); `group_score`: "top2" (the sum of a group's two largest) or "max"; `correction` may be None; `renorm_eps`: the
+    chosen experts' scores are divided by their sum + renorm_eps (None: left as they are)."""
     T = z.shape[0]
     if z.dtype != torch.float32 or z.stride(1) != 1:
         raise QStreamError(QsError.INVALID_INPUT, "moe_route: router logits must be float32 rows")
@@ -745,24 +891,27 @@ def moe_route(z, correction, n_experts, top, groups, keep, scale, gate_col=-1, s
     gate = torch.empty((T,), dtype=torch.float32, device=z.device) if gate_col >= 0 else None
     check(library().qs_moe_route(ptr(idx), ptr(wts), ptr(gate), ptr(z), z.stride(0), ptr(correction), _code(correction), T,
                                  int(n_experts), int(top), int(groups), int(keep), float(scale), int(gate_col),
-                                 {"sigmoid": 0, "softmax": 1}[scores], {"top2": 0, "max": 1}[group_score], stream()))
+                                 {"sigmoid": 0, "softmax": 1}[scores], {"top2": 0, "max": 1}[group_score], -1.0 if renorm_eps is None else float(renorm_eps), stream()))
     return idx, wts, gate
 
 
-def moe_experts_indirect(x, w_up, w_down, idx, wts, tok_slot, activation, add=None, add_scale=None, glu=None) -> torch.Tensor:
+def moe_experts_indirect(x, w_up, w_down, idx, wts, tok_slot, activation, add=None, add_scale=None, glu=None, gated=False) -> torch.Tensor:
     """sum_j wts[t, j] W_down[idx[t, j]] act(W_up[idx[t, j]] x[t]) (+ add[t] * add_scale[t]) in float32 [T, D]; every
     pair finds its expert's matrices (w_up [E, F, D], w_down [E, D, F]) on the device: for steps of few tokens.
     `glu` = (limit, alpha, shift): gated experts, w_up [E, 2 F, D] holding an expert's gate rows above its up rows; the
-    hidden vector is `clamped_glu` of the two halves."""
+    hidden vector is `clamped_glu` of the two halves.  `gated`: w_up likewise, the hidden vector act(gate) * up, taken
+    inside the first kernel."""
     T, D, ldx = _rows(x)
     E, F, _ = w_up.shape
     top = idx.shape[1]
     if w_up.dtype != x.dtype or w_down.dtype != x.dtype or not w_up.is_contiguous() or not w_down.is_contiguous():
         raise QStreamError(QsError.INVALID_INPUT, "experts: matrices and activations must share a type")
+    if gated:
+        F = F // 2
     hidden = torch.empty((T * top, F), dtype=x.dtype, device=x.device)
     out = torch.empty((T, D), dtype=torch.float32, device=x.device)
     check(library().qs_moe_expert_up(ptr(hidden), F, ptr(x), ldx, ptr(w_up), dtype_code(x), _int32(idx, "idx"),
-                                     _int32(tok_slot, "tok_slot"), T, top, D, F, ACTIVATIONS[None if glu else activation], stream()))
+                                     _int32(tok_slot, "tok_slot"), T, top, D, F, ACTIVATIONS[None if glu else activation], int(bool(gated)), stream()))
     if glu:
         hidden = clamped_glu(hidden, *glu)
         F = F // 2

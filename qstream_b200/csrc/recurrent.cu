@@ -16,6 +16,9 @@
 //   gated linear attention with a decay per token and key channel ("gla"):
 //       S_t = diag(w_t) S_{t-1} + k_t v_t^T,   o_t = S_t^T (q_t * q_scale),   w_t = sigmoid(z_t)^decay_scale
 //       (the decay acts before the token's own output, where "wkv" applies it after)
+//   state-space duality, a decay and an input weight per token and head ("ssd"; Mamba-2's recurrence):
+//       S_t = a_t S_{t-1} + b_t k_t v_t^T,   o_t = S_t^T q_t        several heads may share one head of q and k
+//       ("gated" without the normaliser's column)
 //
 // The state lives in 32-bit, per slot as [heads][dv][dk] (a column of S is contiguous), starts at zero and is
 // read at the start of a step and written back at its end; everything between the projections and the output is
@@ -55,7 +58,7 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
                   int H, int dk, int dv, int ks_log2, int cols, int in_act, int vec,
                   const float* __restrict__ ga, const float* __restrict__ gb, size_t ldg, float q_scale, int qk_group,
                   float decay_scale) {
-    constexpr bool WKV = MODE == 1, GATED = MODE == 2, DELTA = MODE == 3, GLA = MODE == 4;
+    constexpr bool WKV = MODE == 1, ONES = MODE == 2, GATED = MODE == 2 || MODE == 5, DELTA = MODE == 3, GLA = MODE == 4, SSD = MODE == 5;
     extern __shared__ float smem[];
     const int KS = 1 << ks_log2, dkp = KS * RK;
     float* sq = smem;                                   // [TILE][dkp]
@@ -64,11 +67,11 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
     float* sv = sw + (WKV || DELTA || GLA ? TILE * dkp : 0);   // [TILE][cols]
     float* carry = sv + TILE * cols;                    // [dkp]         (PHASE 3: the decay from the chunk's start on)
     float* sa = carry + dkp;                            // [TILE]        (GATED: the tokens' decays)
-    const int dvv = GATED ? dv - 1 : dv;                // columns that v holds per head: the gated form adds one of ones
+    const int dvv = ONES ? dv - 1 : dv;                 // columns that v holds per head: the gated form adds one of ones
     grid_dep_launch();
     grid_dep_wait();
     const int s = blockIdx.x, h = blockIdx.y, col0 = blockIdx.z * cols;
-    const int hq = DELTA ? h / qk_group : h;            // the head of q and k that this head reads
+    const int hq = DELTA || SSD ? h / qk_group : h;     // the head of q and k that this head reads
     const int n_cols = min(cols, dv - col0);
     const int tid = threadIdx.x;
     // rows of the packed batch beyond the last sequence belong to nobody: give them a defined value
@@ -164,7 +167,7 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
         if (PHASE != 3) {
             for (int e = tid; e < nt * cols; e += blockDim.x) {
                 const int tt = e / cols, c = e - tt * cols;
-                sv[e] = (c >= n_cols || (DELTA && !v)) ? 0.f : (GATED && col0 + c == dvv) ? 1.0f
+                sv[e] = (c >= n_cols || (DELTA && !v)) ? 0.f : (ONES && col0 + c == dvv) ? 1.0f
                         : apply_activation(to_f32(v[(size_t)(base + tt) * ldv + h * dvv + col0 + c]), in_act);
             }
             if (GATED && tid < nt) sa[tid] = ga[(size_t)(base + tid) * ldg + h];
@@ -477,6 +480,7 @@ int launch_scan(int mode, int phase, float* o, long long ldo, const void* q, lon
         bonus_dtype, state, (size_t)slot_stride, seq_start, seq_slot, n_seq, T_rows, H, dk, dv, ks_log2, cols, in_act, vec, \
         ga, gb, (size_t)ldg, q_scale, qk_group, decay_scale); } while (0)
     if (mode == 3) GO(3, 0);
+    else if (mode == 5) { if (phase == 0) GO(5, 0); else if (phase == 1) GO(5, 1); else GO(5, 3); }
     else if (mode == 4) { if (phase == 0) GO(4, 0); else if (phase == 1) GO(4, 1); else GO(4, 3); }
     else if (mode == 1) { if (phase == 0) GO(1, 0); else if (phase == 1) GO(1, 1); else GO(1, 3); }
     else if (mode == 2) { if (phase == 0) GO(2, 0); else if (phase == 1) GO(2, 1); else GO(2, 3); }
@@ -712,6 +716,7 @@ QS_API int qs_mlstm_output(void* out, int out_dtype, long long ldo, const float*
 namespace {
 }  // namespace
 
+// mode 5: as mode 2 without the column of ones; head h reads head h / qk_group of q and k.
 // mode 2: decay `ga` and input weight `gb` per token and head ([T, H] float32, `ldg` floats between rows), q times
 // `q_scale`; dv counts one column more than v holds (the column of ones that carries the normaliser).
 // mode 0: fixed decay per head (`head_decay` [H], float32 on the device); mode 1: decay exp(-exp(dlog)) per token and
@@ -735,10 +740,10 @@ QS_API int qs_state_scan(int mode, float* o, long long ldo, const void* q, long 
     QS_REQUIRE(dk <= 16 * RK, "state_scan: %d key channels per head above %d", dk, 16 * RK);
     QS_REQUIRE(H <= 65535, "state_scan: %d heads exceed the grid", H);
     QS_REQUIRE(mode == 0 ? head_decay != nullptr : mode == 1 ? (dlog && bonus) : mode == 2 ? (ga && gb && dv > 1)
-               : mode == 4 ? (dlog && decay_scale > 0.f) : (mode == 3 && dlog && gb && !chunk_start),
+               : mode == 5 ? (ga && gb) : mode == 4 ? (dlog && decay_scale > 0.f) : (mode == 3 && dlog && gb && !chunk_start),
                "state_scan: mode %d lacks its operands", mode);
     if (qk_group < 1) qk_group = 1;
-    QS_REQUIRE(mode == 3 ? H % qk_group == 0 : qk_group == 1, "state_scan: %d heads in groups of %d", H, qk_group);
+    QS_REQUIRE(mode == 3 || mode == 5 ? H % qk_group == 0 : qk_group == 1, "state_scan: %d heads in groups of %d", H, qk_group);
     QS_REQUIRE(dtype == QS_F32 || dtype == QS_BF16, "state_scan: unknown dtype %d", dtype);
     const bool wkv = mode == 1 || mode == 4;
     (void)wkv;
@@ -755,7 +760,7 @@ QS_API int qs_state_scan(int mode, float* o, long long ldo, const void* q, long 
     const int n = H * dk;
     chunk_decay_kernel<<<dim3(n_chunks, (n + 127) / 128), 128, 0, stream>>>(chunk_decay, wkv ? dlog : nullptr, (size_t)ldd,
                                                                             head_decay, chunk_start, n, dk,
-                                                                            mode == 2 ? ga : nullptr, (size_t)ldg,
+                                                                            mode == 2 || mode == 5 ? ga : nullptr, (size_t)ldg,
                                                                             mode == 4 ? decay_scale : 0.f);
     if ((rc = qs_check_launch("state_scan chunk decay")) != QS_OK) return rc;
     int by = (int)((per_chunk + 255) / 256);

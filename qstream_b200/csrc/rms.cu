@@ -4,6 +4,9 @@
 //   residual_rmsnorm   x <- x + mult * y (32-bit, in place), and optionally h = rmsnorm(x) in the same pass
 //   branch_norm        x <- x + norm_b(y) * w_b (in place), and optionally h = norm(x) * w in the same pass, with
 //                      norm = layer norm without bias or RMS norm: layers that norm a branch before they add it
+//   stream_tanh_norm   x <- x + sum of up to three branches (32-bit, in place), each with a factor and, if it has a
+//                      weight, divided by its root mean square first; then up to two reads of the new x in the same
+//                      pass: tanh(alpha x) * w + b (no statistics), or x itself
 //   gated_group_norm   out = o / sqrt(mean_group(o^2) + eps) * w * act(gate), groups of consecutive elements
 //                      (one group = the whole row, or one per head; group 0 = no norm, only the gate)
 //   gated_act          out = act(a) * b for the two halves [a | b] of a fused projection (gated feed-forward)
@@ -130,6 +133,86 @@ int launch_branch_norm(void* h_out, long long ldh, void* x, long long ldx, const
                                         (size_t)ldx, (const TY*)y, (size_t)ldy, wy, wy_dtype, w, w_dtype, D, eps, center);
     if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "branch_norm: %s", cudaGetErrorString(e));
     return qs_check_launch("branch_norm");
+}
+
+// ----------------------------------------------------------------------------- branches into the stream, tanh norms
+
+struct StreamBranch { const float* y; size_t ld; const void* w; int w_dtype; float mult; };
+struct TanhRead { void* h; size_t ld; const void* w; const void* b; int w_dtype, b_dtype; float alpha; };
+
+// One block per row; V neighbouring columns per thread and round (V = 4: 16-byte aligned rows of whole fours).  The
+// sums of squares of the normed branches are taken together.  A read without a weight hands on x itself.
+template <typename TH, int V>
+__global__ void stream_tanh_norm_kernel(float* __restrict__ x, size_t ldx, StreamBranch b0, StreamBranch b1, StreamBranch b2, TanhRead r0,
+                                        TanhRead r1, int D, float eps) {
+    __shared__ float part[3][32];
+    grid_dep_launch();
+    grid_dep_wait();
+    const size_t t = blockIdx.x;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+    const StreamBranch br[3] = {b0, b1, b2};
+    float scale[3] = {b0.mult, b1.mult, b2.mult};
+    if (b0.w || b1.w || b2.w) {
+        float q[3] = {0.f, 0.f, 0.f};
+        for (int i = threadIdx.x * V; i < D; i += blockDim.x * V)
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+                if (br[k].w)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) { const float y = br[k].y[t * br[k].ld + i + v]; q[k] = fmaf(y, y, q[k]); }
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            q[k] = warp_sum(q[k]);
+            if (lane == 0) part[k][warp] = q[k];
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 3; ++k)
+            if (br[k].w) {
+                float total = 0.f;
+                for (int i = 0; i < warps; ++i) total += part[k][i];
+                scale[k] *= 1.0f / sqrtf(total / (float)D + eps);
+            }
+    }
+    float* xr = x + t * ldx;
+    for (int i = threadIdx.x * V; i < D; i += blockDim.x * V) {
+        float xv[V];
+#pragma unroll
+        for (int v = 0; v < V; ++v) xv[v] = xr[i + v];
+        if (b0.y) {
+            float add[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) add[v] = 0.f;
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+                if (br[k].y)
+#pragma unroll
+                    for (int v = 0; v < V; ++v) {
+                        const float y = br[k].y[t * br[k].ld + i + v] * scale[k];
+                        add[v] += br[k].w ? y * load_as_f32(br[k].w, br[k].w_dtype, i + v) : y;
+                    }
+#pragma unroll
+            for (int v = 0; v < V; ++v) { xv[v] += add[v]; xr[i + v] = xv[v]; }
+        }
+        const TanhRead rd[2] = {r0, r1};
+#pragma unroll
+        for (int k = 0; k < 2; ++k)
+            if (rd[k].h) {
+                float h[V];
+#pragma unroll
+                for (int v = 0; v < V; ++v)
+                    h[v] = rd[k].w ? fmaf(tanhf(rd[k].alpha * xv[v]), load_as_f32(rd[k].w, rd[k].w_dtype, i + v), load_as_f32(rd[k].b, rd[k].b_dtype, i + v))
+                                   : xv[v];
+                TH* dst = reinterpret_cast<TH*>(rd[k].h) + t * rd[k].ld + i;
+                if (V == 4 && sizeof(TH) == 2) {
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(h[0], h[1 % V]), hi = __floats2bfloat162_rn(h[2 % V], h[3 % V]);
+                    *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+                } else {
+#pragma unroll
+                    for (int v = 0; v < V; ++v) dst[v] = from_f32<TH>(h[v]);
+                }
+            }
+    }
 }
 
 // ----------------------------------------------------------------------------- gated group norm
@@ -353,6 +436,35 @@ QS_API int qs_branch_norm(void* h_out, int h_dtype, long long ldh, void* x, int 
     if (x_dtype == QS_BF16 && y_dtype == QS_BF16 && h_dtype == QS_BF16) GO(bf16, bf16, bf16);
 #undef GO
     return qs_fail(QS_ERR_INVALID_INPUT, "branch_norm: unsupported types x=%d y=%d h=%d", x_dtype, y_dtype, h_dtype);
+}
+
+// x [rows, D] float32 (row stride ldx).  Branches y0..y2 float32 or null (a null one ends the list), with factors m0..m2
+// and, for a branch that is divided by its root mean square over D first, a weight w0..w2.  Reads h0, h1 (null: none) of
+// type `h_dtype`: tanh(alpha x) * w + b, or, with a null weight, x.
+QS_API int qs_stream_tanh_norm(float* x, long long ldx, int rows, int D, float eps, const float* y0, long long ld0, float m0, const void* w0,
+                               int w0_dtype, const float* y1, long long ld1, float m1, const void* w1, int w1_dtype, const float* y2,
+                               long long ld2, float m2, const void* w2, int w2_dtype, int h_dtype, void* h0, long long ldh0, float alpha0,
+                               const void* nw0, int nw0_dtype, const void* nb0, int nb0_dtype, void* h1, long long ldh1, float alpha1,
+                               const void* nw1, int nw1_dtype, const void* nb1, int nb1_dtype, cudaStream_t stream) {
+    if (rows == 0) return QS_OK;
+    QS_REQUIRE(rows > 0 && D > 0 && x, "stream_tanh_norm: bad sizes");
+    QS_REQUIRE((y0 || !y1) && (y1 || !y2), "stream_tanh_norm: a branch behind a missing one");
+    QS_REQUIRE((!w0 || y0) && (!w1 || y1) && (!w2 || y2), "stream_tanh_norm: a weight without its branch");
+    QS_REQUIRE((!nw0 || (h0 && nb0)) && (!nw1 || (h1 && nb1)), "stream_tanh_norm: a norm lacks its output or its shift");
+    QS_REQUIRE(h_dtype == QS_F32 || h_dtype == QS_BF16, "stream_tanh_norm: unknown dtype %d", h_dtype);
+    const StreamBranch b0 = {y0, (size_t)ld0, w0, w0_dtype, m0}, b1 = {y1, (size_t)ld1, w1, w1_dtype, m1}, b2 = {y2, (size_t)ld2, w2, w2_dtype, m2};
+    const TanhRead r0 = {h0, (size_t)ldh0, nw0, nb0, nw0_dtype, nb0_dtype, alpha0}, r1 = {h1, (size_t)ldh1, nw1, nb1, nw1_dtype, nb1_dtype, alpha1};
+    auto fits = [](const void* p, long long ld) { return !p || (((uintptr_t)p % 16) == 0 && ld % 4 == 0); };
+    const bool vec = D % 4 == 0 && fits(x, ldx) && fits(y0, ld0) && fits(y1, ld1) && fits(y2, ld2) && fits(h0, ldh0) && fits(h1, ldh1);
+    const int items = vec ? (D + 3) / 4 : D;
+    const int threads = items >= 512 ? 512 : (items >= 256 ? 256 : 128);
+    cudaError_t e;
+#define GO(TH, V) e = qs_launch_dependent(stream_tanh_norm_kernel<TH, V>, dim3(rows), dim3(threads), 0, stream, x, (size_t)ldx, b0, b1, b2, r0, r1, D, eps)
+    if (h_dtype == QS_F32) { if (vec) GO(float, 4); else GO(float, 1); }
+    else { if (vec) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
+#undef GO
+    if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "stream_tanh_norm: %s", cudaGetErrorString(e));
+    return qs_check_launch("stream_tanh_norm");
 }
 
 QS_API int qs_gated_group_norm(void* out, int out_dtype, long long ldo, const void* o, int o_dtype, long long ldi,

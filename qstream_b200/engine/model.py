@@ -40,6 +40,8 @@ def _part_declarations(spec: ModelSpec):
     for block in spec.layers:
         for role, ps in part_class("arrangement", block.arrangement).part_specs(block):
             yield ps, part_class(role, ps.kind).declare(ps)
+    for joint in getattr(spec, "joints", ()):
+        yield joint, part_class("joint", joint.kind).declare(joint)
     if spec.final_norm is not None:
         yield spec.final_norm, part_class("norm", spec.final_norm.kind).declare(spec.final_norm)
     yield spec.head, part_class("head", spec.head.kind).declare(spec.head)
@@ -79,6 +81,7 @@ class CausalLM:
 
         self.embedding = make("embedding", spec.embedding)
         self.blocks = [build_block(b, tensors_of, self.runtime) for b in spec.layers]
+        self.joints = [make("joint", j) for j in getattr(spec, "joints", ())]
         self.final_norm = make("norm", spec.final_norm) if spec.final_norm is not None else None
         self.head = make("head", spec.head)
         if getattr(spec.head, "tied", False):
@@ -126,6 +129,8 @@ class CausalLM:
         for i, run in enumerate(self.spec.schedule):
             if not 0 <= run.layer < len(self.blocks):
                 raise QStreamError(QsError.INVALID_MODEL, f"schedule entry {i} names layer {run.layer}")
+            if run.enter is not None and not 0 <= run.enter[0] < len(self.joints):
+                raise QStreamError(QsError.INVALID_MODEL, f"schedule entry {i} names joint {run.enter[0]}")
             parts = self.blocks[run.layer].cached_parts()
             ids = run.cache if isinstance(run.cache, (tuple, list)) else (run.cache,)
             if len(ids) != len(parts):
@@ -171,8 +176,12 @@ class CausalLM:
         if record is not None:
             ops.check_finite(x, n_runs, record, b.tok_slot)
         settle = getattr(step, "settle", lambda t: t)
+        for joint in self.joints:
+            joint.begin(x, step)
         for i, run in enumerate(self.spec.schedule):
             block = self.blocks[run.layer]
+            if run.enter is not None:                       # a step of the model's own before this run (a loop's next pass)
+                x = self.joints[run.enter[0]].forward(x, step, run.enter[1])
             if not getattr(block, "takes_pending", False):
                 x = settle(x)                               # a layer that wants the stream with nothing left to add
             x = block.forward(x, step, run.cache)

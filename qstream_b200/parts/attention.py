@@ -9,7 +9,8 @@ three projections are one matrix product over the concatenated weights.
 Options a spec may switch on, each with its constants as the spec's fields: values with a head size of
 their own; a factor on the scores other than head_dim^-1/2; a tanh cap on the scores; values blended
 with those that an earlier layer computed for the same token (what is cached is the blend); a sigmoid gate
-from the mixer's input on the concatenated heads (its projection rides in the same product as q, k, v); keys seen
+from the mixer's input on the concatenated heads, a value per channel or per head (its projection rides in the same
+product as q, k, v); keys seen
 only inside the query's chunk of positions, or inside a window that also keeps the sequence's first tokens; a learned
 sink per head in the softmax's denominator; two attention maps per head over the same values, joined as a difference
 with a unit RMS per head (differential attention); one RMS norm over the whole q and the whole k projection before the
@@ -54,7 +55,7 @@ class Attention(Mixer):
                 d["k_bias"] = TensorDecl((hkv,), "bias")
                 d["v_bias"] = TensorDecl((hv,), "bias")
         if spec.gate:
-            d["gate"] = TensorDecl((ho, spec.width))
+            d["gate"] = TensorDecl((spec.n_heads if spec.gate == "head" else ho, spec.width))
         if spec.value_mix is not None:
             d["value_mix"] = TensorDecl((), "fraction")
         if spec.out_bias:
@@ -79,6 +80,11 @@ class Attention(Mixer):
             raise QStreamError(QsError.INVALID_MODEL, "attention: values taken from the keys have the keys' size, no bias and no blend")
         names = ["q"] if spec.shares_cache else (["q", "k"] if self.values_from_keys else ["q", "k", "v"])
         mats = [tensors[n] for n in names] + ([tensors["gate"]] if spec.gate else [])
+        self.gate_rows = tensors["gate"].shape[0] if spec.gate else 0
+        self.gate_at = sum(m.shape[0] for m in mats) - self.gate_rows       # the gate's first column of the product
+        pad = -sum(m.shape[0] for m in mats) % 8 if spec.gate == "head" else 0
+        if pad:                                         # rows of zeros, so that the product's rows stay 16-byte aligned
+            mats.append(torch.zeros((pad, spec.width), dtype=mats[0].dtype, device=mats[0].device))
         if len({m.dtype for m in mats}) != 1:
             raise QStreamError(QsError.INVALID_MODEL, "q/k/v projections are stored in different types")
         self.w_qkv = torch.cat(mats, dim=0).contiguous() if len(mats) > 1 else mats[0]
@@ -86,7 +92,7 @@ class Attention(Mixer):
         if spec.qkv_bias:
             biases = [tensors[n + "_bias"].float() for n in names]
             if spec.gate:                               # the gate's rows of the product have no bias
-                biases.append(torch.zeros(tensors["gate"].shape[0], dtype=torch.float32, device=biases[0].device))
+                biases.append(torch.zeros(self.gate_rows + pad, dtype=torch.float32, device=biases[0].device))
             self.b_qkv = torch.cat(biases).contiguous()
         # the blend's weight is a constant of the model: read once, passed to the kernel by value
         self.value_mix = float(tensors["value_mix"].float().item()) if spec.value_mix == "blend" else 0.0
@@ -192,7 +198,7 @@ class Attention(Mixer):
                            b.tok_slot, b.tok_pos, view.page_table, view.page_tokens, view.k, view.v,
                            step.status, settled=True,     # a step's slots, positions and pages arrive before its first kernel
                            v_head_dim=s.value_dim, v_first=v_first, v_mix=self.value_mix, half_layout=half)
-        gate = qkv[:, qkv.shape[1] - s.n_heads * s.value_dim:] if s.gate else None
+        gate = qkv[:, self.gate_at:self.gate_at + self.gate_rows] if s.gate else None
         if not self.masked:
             return attend(q, s, step, view, out, gate=gate)
         return self._attend_masked(q, step, view, out, gate)
@@ -218,7 +224,7 @@ class Attention(Mixer):
         if two:
             o = ops.pair_diff_norm(o, s.n_heads, s.value_dim, self.lam, 1.0 - float(s.diff), float(s.eps), q.dtype)
         if gate is not None:
-            o = ops.gated_group_norm(o, 0, None, gate, "sigmoid", 0.0, o.dtype)
+            o = ops.gated_group_norm(o, 0, None, gate, "sigmoid", 0.0, o.dtype, gate_span=s.value_dim if s.gate == "head" else 1)
         if out is not None and o.data_ptr() != out.data_ptr():
             out.copy_(o)
             return out
@@ -227,8 +233,8 @@ class Attention(Mixer):
 
 def attend(q, spec, step, view, out=None, gate=None, sink=None):
     """Pick the attention kernel for this step: decode and prefill have their own
-    bfloat16 kernels; the generic kernel takes every other case.  `gate` [T, heads * value_dim]: the result
-    times sigmoid(gate), in the bfloat16 kernels' last stage or by a kernel of its own.  `sink` (float32, one per
+    bfloat16 kernels; the generic kernel takes every other case.  `gate` [T, heads * value_dim] ([T, heads] where the
+    spec's gate is "head"): the result times sigmoid(gate), in the bfloat16 kernels' last stage or by a kernel of its own.  `sink` (float32, one per
     query head): exp(sink) joins each softmax's denominator."""
     b = step.batch
     if q.dtype == torch.bfloat16:
@@ -240,7 +246,7 @@ def attend(q, spec, step, view, out=None, gate=None, sink=None):
                       b.tok_slot, b.tok_pos, view.page_table, view.page_tokens, view.k, view.v,
                       step.status, out=out, v_head_dim=spec.value_dim, softcap=spec.softcap, sink=sink)
     if gate is not None:
-        o = ops.gated_group_norm(o, 0, None, gate, "sigmoid", 0.0, o.dtype)
+        o = ops.gated_group_norm(o, 0, None, gate, "sigmoid", 0.0, o.dtype, gate_span=spec.value_dim if spec.gate == "head" else 1)
     return o
 
 

@@ -303,6 +303,112 @@ class PostNormBlock(Arrangement):
         return x
 
 
+class PendingBranches:
+    """Branches that are still to be added to the 32-bit stream, each with a factor and perhaps the weight of a norm it
+    passes first: x += sum of factor * branch.  Whoever reads x next adds them in the same kernel."""
+
+    def __init__(self, branches, eps):
+        self.branches, self.eps = branches, eps
+
+    def apply(self, x):
+        from ..csrc import ops
+        ops.stream_tanh_norm(x, self.branches, self.eps)
+        return x
+
+
+class TwinNormBlock(Arrangement):
+    """Both sublayers read the same x through a norm each: x += mixer(norm_1(x)) + ffn(norm_2(x)), with the residual stream
+    x in 32-bit whatever the engine's type and updated in place; a layer may have no feed-forward.  The branches arrive
+    in 32-bit from their last product and stay pending (`step.pending`): adding them to x (a mixer that offers
+    `normed_branches` leaves its results' norms to that kernel too) and the two norms of the next layer's read are one kernel.
+    Norms that offer `tanh_read` (the dynamic tanh) are taken in that kernel, others behind it."""
+    norm_names = ("input",)
+    takes_pending = True
+
+    def __init__(self, spec, parts, runtime):
+        super().__init__(spec, parts, runtime)
+        import inspect
+        import torch
+        if self.ffn is not None and "ffn_input" not in self.norms:
+            raise QStreamError(QsError.INVALID_MODEL, "a twin-norm layer with a feed-forward needs the norm 'ffn_input'")
+        self.wide = torch.float32
+        self._typed = {id(p): "out_dtype" in inspect.signature(p.forward).parameters for p in (self.mixer, self.ffn) if p}
+        self.eps = float(getattr(self.mixer.spec, "eps", 0.0))          # of the norms that a pair's results pass
+        self.reads = [self.norms["input"]] + ([self.norms["ffn_input"]] if self.ffn is not None else [])
+
+    part_specs = classmethod(ScaledResidualBlock.part_specs.__func__)      # a layer may lack its feed-forward here too
+    build = classmethod(ScaledResidualBlock.build.__func__)
+
+    def cached_parts(self):
+        return getattr(self.mixer, "cached_parts", lambda: [self.mixer])()
+
+    def _branch(self, part, *args):
+        from ..csrc import ops
+        y = part.forward(*args, **({"out_dtype": self.wide} if self._typed[id(part)] else {}))
+        return (1.0, y if y.dtype == self.wide else ops.convert(y, self.wide), None)
+
+    def forward(self, x, step, cache_id):
+        from ..csrc import ops
+        before, step.pending = step.pending, None
+        if all(hasattr(n, "tanh_read") for n in self.reads):
+            if before is not None and not isinstance(before, PendingBranches):
+                x, before = before.apply(x), None
+            branches, eps = (before.branches, before.eps) if before is not None else ((), 0.0)
+            hs = ops.stream_tanh_norm(x, branches, eps, [n.tanh_read() for n in self.reads], self.runtime.dtype)
+        else:
+            x = before.apply(x) if before is not None else x
+            hs = [n.forward(x) for n in self.reads]
+        if hasattr(self.mixer, "normed_branches"):
+            ys = self.mixer.normed_branches(hs[0], step, cache_id, out_dtype=self.wide)
+        else:
+            ys = [self._branch(self.mixer, hs[0], step, cache_id)]
+        if self.ffn is not None:
+            ys.append(self._branch(self.ffn, hs[1], step))
+        step.pending = PendingBranches(ys, self.eps)
+        return x
+
+
+class LoopEntry(Part):
+    """Before each pass of a looped group of layers: x <- W_in [x; x0] + step[t], x0 the embedding's output.  x (with what
+    is still pending) and x0 lie side by side in one buffer in the engine's type, x0 written once a step; the product's
+    result, the pass's vector added on its accumulator, is the new 32-bit stream."""
+    role = "joint"
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        from ..weights.loader import TensorDecl
+        return {"in": TensorDecl((spec.width, 2 * spec.width)), "step": TensorDecl((spec.times, spec.width), "bias")}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.w_in = tensors["in"]
+        self.steps = [row.clone() for row in tensors["step"].float()]
+
+    def begin(self, x, step):
+        import torch
+        from ..csrc import ops
+        D = self.spec.width
+        both = torch.empty((x.shape[0], 2 * D), dtype=self.runtime.dtype, device=x.device)
+        wide = x if x.dtype == torch.float32 else ops.convert(x, torch.float32)
+        ops.stream_tanh_norm(wide, reads=[(0.0, None, None, both[:, D:])], out_dtype=both.dtype)
+        step.scratch[id(self)] = both
+
+    def forward(self, x, step, t):
+        import torch
+        from ..csrc import ops
+        from .linear import linear
+        both, D = step.scratch[id(self)], self.spec.width
+        branches, eps = (), 0.0
+        if isinstance(step.pending, PendingBranches):
+            branches, eps, step.pending = step.pending.branches, step.pending.eps, None
+        else:
+            x = step.settle(x)
+        wide = x if x.dtype == torch.float32 else ops.convert(x, torch.float32)
+        ops.stream_tanh_norm(wide, branches, eps, [(0.0, None, None, both[:, :D])], both.dtype)
+        return linear(both, self.w_in, self.steps[t], out_dtype=torch.float32)
+
+
 class HyperConnection(Part):
     """The tensors with which one sublayer meets a residual stream kept in several copies: the weights of the read
     (`in`), of the write (`out`), the matrix that mixes the copies (`mix`, [from, to]) and the vector that scales the
@@ -426,6 +532,8 @@ class HyperBlock(Arrangement):
         return x
 
 
+register("arrangement", "twin_norm", TwinNormBlock)
+register("joint", "loop_entry", LoopEntry)
 register("arrangement", "hyper", HyperBlock)
 register("connection", "hyper_connection", HyperConnection)
 register("arrangement", "parallel", ParallelBlock)

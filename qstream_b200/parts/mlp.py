@@ -86,7 +86,9 @@ class RoutedExperts(FeedForward):
     experts of the best groups (csrc/moe.cu), their outputs are added with the router's weights in 32-bit, and an
     optional shared expert runs for every token, multiplied by a sigmoid gate of its own.  The router's logits are
     a product with 32-bit sums and a 32-bit result; the shared gate's row rides in the same product.  Options of the
-    spec: softmax scores, a group's score as its largest, no correction, an ungated shared expert, and gated experts
+    spec: softmax scores, a group's score as its largest, no correction, weights made to sum to one, an ungated shared
+    expert, experts act(gate) * up (an expert's gate rows stacked above its up rows; the unit inside the first kernel where
+    the pairs go through the routing table, a kernel of its own behind the products), and clamped gated experts
     (an expert's gate rows stacked above its up rows in one matrix; the clamped gated unit is a kernel of its own
     between the two products)."""
     captures_any_step = False           # a step with many tokens reads the experts' row counts on the host
@@ -116,13 +118,16 @@ class RoutedExperts(FeedForward):
         if spec.activation not in ops.ACTIVATIONS:
             raise QStreamError(QsError.UNSUPPORTED_ARCH, f"activation '{spec.activation}' has no kernel")
         E = spec.n_experts
-        self.gated = bool(getattr(spec, "gated", False))
+        self.gated = getattr(spec, "gated", False)
+        if self.gated not in (False, True, "act") or (self.gated == "act" and spec.shared_inner):
+            raise QStreamError(QsError.UNSUPPORTED_ARCH, f"routed experts: gated '{self.gated}' with a shared expert of {spec.shared_inner}")
+        self.renorm_eps = float(spec.normalize_eps) if getattr(spec, "normalize", False) else None
         self.scores, self.group_score = getattr(spec, "scores", "sigmoid"), getattr(spec, "group_score", "top2")
         if self.scores not in ("sigmoid", "softmax") or self.group_score not in ("top2", "max"):
             raise QStreamError(QsError.UNSUPPORTED_ARCH, f"routed experts: scores '{self.scores}', group score '{self.group_score}'")
         # (limit, alpha, shift) of the clamped gated unit, for the routed experts and for the shared one
-        self.glu = (float(spec.limit), float(spec.glu_alpha), float(spec.glu_shift)) if self.gated else None
-        self.shared_glu = (float(spec.shared_limit), float(spec.glu_alpha), float(spec.glu_shift)) if self.gated else None
+        self.glu = (float(spec.limit), float(spec.glu_alpha), float(spec.glu_shift)) if self.gated is True else None
+        self.shared_glu = (float(spec.shared_limit), float(spec.glu_alpha), float(spec.glu_shift)) if self.gated is True else None
         if self.gated:                                  # an expert's gate rows above its up rows: one product for both
             self.w_up = torch.stack([torch.cat([tensors[f"gate{e}"], tensors[f"up{e}"]], dim=0) for e in range(E)]).contiguous()
         else:
@@ -144,14 +149,15 @@ class RoutedExperts(FeedForward):
         z = linear(h, self.w_router, out_dtype=torch.float32)
         idx, wts, gate = ops.moe_route(z, self.correction, s.n_experts, s.top, s.groups, s.keep, s.route_scale,
                                        gate_col=s.n_experts if self.shared_gate else -1, scores=self.scores,
-                                       group_score=self.group_score)
+                                       group_score=self.group_score, renorm_eps=self.renorm_eps)
         shared = None
         if self.shared and self.gated:
             shared = linear(ops.clamped_glu(linear(h, self.shared_up), *self.shared_glu), self.shared_down, out_dtype=torch.float32)
         elif self.shared:
             shared = linear(linear(h, self.shared_up, activation=s.activation), self.shared_down, out_dtype=torch.float32)
         if b.decode or h.shape[0] <= INDIRECT_ROWS:
-            out = ops.moe_experts_indirect(h, self.w_up, self.w_down, idx, wts, b.tok_slot, s.activation, shared, gate, glu=self.glu)
+            out = ops.moe_experts_indirect(h, self.w_up, self.w_down, idx, wts, b.tok_slot, s.activation, shared, gate, glu=self.glu,
+                                           gated=self.gated == "act")
         else:
             offsets, place_token, pair_place = ops.moe_sort(idx, s.n_experts)
             rows = ops.gather_rows(h, place_token)
@@ -159,8 +165,10 @@ class RoutedExperts(FeedForward):
             y = torch.empty((rows.shape[0], s.width), dtype=torch.float32, device=h.device)
             bounds = offsets.tolist()                   # waits for the device: how many rows each expert got
             ops.expert_products(hidden, rows, self.w_up, bounds)        # a product per expert, launched by one call
-            if self.gated:
-                hidden = ops.clamped_glu(hidden, *self.glu)             # one launch for all experts' rows
+            if self.gated == "act":
+                hidden = ops.gated_act(hidden, s.activation)            # one launch for all experts' rows
+            elif self.gated:
+                hidden = ops.clamped_glu(hidden, *self.glu)
             else:
                 ops.activate(hidden, s.activation)
             ops.expert_products(y, hidden, self.w_down, bounds)

@@ -1,6 +1,6 @@
 """LayerNorm with weight and optional bias (QStream src/kernels_scalar.c:151-171), and the RMS norm
 x / sqrt(mean(x^2) + eps) * (offset + weight) (the reference's `rmsnorm`, src/kernels_scalar.c:173-186, has
-offset 0; weights stored around zero take offset 1)."""
+offset 0; weights stored around zero take offset 1); the dynamic tanh, which stands in a norm's place."""
 from __future__ import annotations
 
 from ..csrc import ops
@@ -113,7 +113,34 @@ class StreamSumNorm(Norm):
                                   out_dtype=self.runtime.dtype)
 
 
+class TanhNorm(Norm):
+    """The dynamic tanh: tanh(alpha x) * weight + shift, no statistics; reads the 32-bit stream and writes the engine's type.
+    `tanh_read()` is what `ops.stream_tanh_norm` takes, so that an arrangement can add branches to the stream and read it
+    through one or two such norms in one pass."""
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        return {"weight": TensorDecl((spec.size,), "norm_weight"), "shift": TensorDecl((spec.size,), "bias"),
+                "alpha": TensorDecl((), "norm_weight")}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.weight, self.shift = tensors["weight"], tensors["shift"]
+        self.alpha = float(tensors["alpha"].float().item())     # a constant of the model: read once, passed by value
+
+    def tanh_read(self):
+        return self.alpha, self.weight, self.shift, None
+
+    def forward(self, x):
+        import torch
+        if x.dtype != torch.float32:
+            x = ops.convert(x, torch.float32)
+        return ops.stream_tanh_norm(x, reads=[self.tanh_read()], out_dtype=self.runtime.dtype)[0]
+
+
 register("norm", "layernorm", LayerNorm)
+register("norm", "tanh_norm", TanhNorm)
 register("norm", "stream_sum_rmsnorm", StreamSumNorm)
 register("norm", "stream_norm", StreamNorm)
 register("norm", "rmsnorm", RmsNorm)

@@ -16,6 +16,13 @@ then a silu gate and W_o.
 `GatedDelta` ("gated_delta"): the delta rule with a decay per token, head and key channel and a step size per token
 and head, behind short causal convolutions on q, k and v.  `PairMixer` ("pair"): two mixers side by side.
 
+`Mamba2` ("mamba2"): the state-space dual form, a decay and a step size per token and head, B and C shared by groups of
+heads, a short convolution in front, a gate before the norm.
+
+With a state per channel instead of a matrix per head (csrc/channel.cu), behind a short causal convolution:
+`Mamba` ("mamba"): the selective scan, several states per channel with a decay per token, channel and state;
+`RgLru` ("rglru"): the real-gated linear recurrent unit, one state per channel.
+
 All keep S in 32-bit per sequence (`StateNeed`), zero when a slot is taken, read at the start of a step and
 written at its end by one kernel that walks a sequence's tokens in order (csrc/recurrent.cu); single tokens and
 short prompts take that path, a long prompt is cut into chunks that run side by side and are joined by a prefix
@@ -292,16 +299,168 @@ class GatedDelta(Mixer):
         return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
 
 
+LOG2E = 1.4426950408889634
+
+
+def _conv_state(taps, channels, dtype):
+    return {"conv": StateNeed((taps - 1, channels), dtype)} if taps > 1 else {}
+
+
+def run_short_conv(x, taps, bias, step, cache_id, activation):
+    """The short convolution of a mixer's channels, with the inputs that earlier steps left under the state "conv"."""
+    b = step.batch
+    held = step.state(cache_id, "conv") if taps.shape[1] > 1 else None
+    out = ops.short_conv(x, taps, bias, held, b.tok_slot, b.tok_pos, activation, decode=b.decode)
+    if held is not None and not b.decode:                   # after the convolution has read it
+        ops.conv_keep(held, x, b.seq_start, b.seq_slot, b.n_seq)
+    return out
+
+
+class Mamba(Mixer):
+    """The selective scan.  W_in is one product; the convolution and silu one kernel; W_x (the step sizes' low-rank input, B
+    and C) and W_dt (32-bit results, its bias in the product) a product each; the scan takes the softplus, the decays, D x
+    and the silu gate, all in 32-bit (a long prompt: its chunks side by side, joined by a prefix over the chunks' states)."""
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        D, n, N, R = spec.width, spec.inner, spec.state, spec.dt_rank
+        return {"in": TensorDecl((2 * n, D)), "conv": TensorDecl((n, spec.conv_taps)), "conv_bias": TensorDecl((n,), "bias"),
+                "x": TensorDecl((R + 2 * N, n)), "dt": TensorDecl((n, R)), "dt_bias": TensorDecl((n,), "bias"),
+                "A_log": TensorDecl((n, N), "bias"), "D": TensorDecl((n,), "norm_weight"), "o": TensorDecl((D, n))}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        if spec.state > 512:
+            raise QStreamError(QsError.UNSUPPORTED_ARCH, f"mamba: {spec.state} states per channel (the kernel takes up to 512)")
+        self.w_in, self.w_x, self.w_dt, self.w_out = tensors["in"], tensors["x"], tensors["dt"], tensors["o"]
+        self.conv, self.conv_bias = tensors["conv"].contiguous(), tensors["conv_bias"]
+        self.dt_bias, self.d = tensors["dt_bias"].float().contiguous(), tensors["D"].float().contiguous()
+        self.a2 = (tensors["A_log"].double().exp() * -LOG2E).float().contiguous()       # A log2(e): the kernel takes powers of two
+
+    def state_need(self):
+        s = self.spec
+        return {"channels": StateNeed((s.inner, s.state), torch.float32), **_conv_state(s.conv_taps, s.inner, self.runtime.dtype)}
+
+    def forward(self, h, step, cache_id, residuals=(), out_dtype=None):
+        s, b = self.spec, step.batch
+        n, R, N = s.inner, s.dt_rank, s.state
+        p = linear(h, self.w_in)
+        x = run_short_conv(p[:, :n], self.conv, self.conv_bias, step, cache_id, "silu")
+        low = linear(x, self.w_x)
+        raw = linear(low[:, :R], self.w_dt, self.dt_bias, out_dtype=torch.float32)
+        y = ops.selective_scan(x, raw, self.a2, low[:, R:R + N], low[:, R + N:], self.d, p[:, n:], step.state(cache_id, "channels"),
+                               b.seq_start, b.seq_slot, b.n_seq, chunks=scan_chunks(b, h.device))
+        return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
+
+
+# A step of at most this many rows takes a block-diagonal product as one launch for all blocks.
+FEW_TOKENS = 32
+
+
+class RgLru(Mixer):
+    """Griffin's recurrent block.  Both branches are one product (biases in it); the convolution one kernel; the two gates of
+    every block of channels one product per block with 32-bit results (all blocks in one launch for few tokens); the scan
+    takes the gates' biases and sigmoids, the decays, the recurrence, and the gelu of the other branch, in 32-bit."""
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        D, n, nb = spec.width, spec.inner, spec.blocks
+        k = n // nb
+        d = {"conv": TensorDecl((n, spec.conv_taps)), "conv_bias": TensorDecl((n,), "bias"), "lam": TensorDecl((n,), "bias"),
+             "o": TensorDecl((D, n))}
+        for name in ("y", "x"):
+            d.update({name: TensorDecl((n, D)), name + "_bias": TensorDecl((n,), "bias")})
+        for name in ("r", "i"):
+            d.update({name: TensorDecl((nb, k, k)), name + "_bias": TensorDecl((nb, k), "bias")})
+        return d
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        if spec.inner % spec.blocks:
+            raise QStreamError(QsError.INVALID_MODEL, f"rglru: {spec.inner} channels in {spec.blocks} blocks")
+        self.w_in = torch.cat([tensors["y"], tensors["x"]], dim=0).contiguous()
+        self.b_in = torch.cat([tensors["y_bias"].float(), tensors["x_bias"].float()]).contiguous()
+        self.conv, self.conv_bias = tensors["conv"].contiguous(), tensors["conv_bias"]
+        self.w_gates = torch.cat([tensors["r"], tensors["i"]], dim=1).contiguous()             # [blocks, 2 k, k]
+        self.b_gates = torch.cat([tensors["r_bias"].float(), tensors["i_bias"].float()], dim=1).reshape(-1).contiguous()
+        self.rate = (8.0 * torch.nn.functional.softplus(tensors["lam"].double())).float().contiguous()
+        self.w_out = tensors["o"]
+
+    def state_need(self):
+        s = self.spec
+        return {"channels": StateNeed((s.inner,), torch.float32), **_conv_state(s.conv_taps, s.inner, self.runtime.dtype)}
+
+    def forward(self, h, step, cache_id, residuals=(), out_dtype=None):
+        s, b = self.spec, step.batch
+        n = s.inner
+        p = linear(h, self.w_in, self.b_in)
+        u = run_short_conv(p[:, n:], self.conv, self.conv_bias, step, cache_id, None)
+        gates = torch.empty((h.shape[0], 2 * n), dtype=torch.float32, device=h.device)
+        (ops.head_linear if h.shape[0] <= FEW_TOKENS else ops.head_products)(gates, u, self.w_gates, s.blocks)
+        y = ops.gated_lru(u, gates, self.b_gates, self.rate, p[:, :n], step.state(cache_id, "channels"), n // s.blocks,
+                          b.seq_start, b.seq_slot, b.n_seq, chunks=scan_chunks(b, h.device))
+        return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
+
+
+class Mamba2(Mixer):
+    """Mamba-2.  z, x, B and C are one product in the engine's type, the step sizes one with a 32-bit result; the convolution
+    and silu one kernel; the decays and step sizes one (32-bit); the matrix scan of the other mixers in its "ssd" form (C
+    as q, B as k, x as v; a long prompt in chunks side by side); D x, the gate and the norm over parts one kernel."""
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        D, n, H, GN = spec.width, spec.inner, spec.n_heads, spec.groups * spec.state
+        return {"in": TensorDecl((2 * n + 2 * GN + H, D)), "conv": TensorDecl((n + 2 * GN, spec.conv_taps)),
+                "conv_bias": TensorDecl((n + 2 * GN,), "bias"), "dt_bias": TensorDecl((H,), "bias"), "A_log": TensorDecl((H,), "bias"),
+                "D": TensorDecl((H,), "norm_weight"), "norm": TensorDecl((n,), "norm_weight"), "o": TensorDecl((D, n))}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        if spec.n_heads % spec.groups or spec.inner % spec.norm_parts:
+            raise QStreamError(QsError.INVALID_MODEL, f"mamba2: {spec.n_heads} heads in {spec.groups} groups, {spec.inner} channels in {spec.norm_parts} parts")
+        if spec.state > 256:
+            raise QStreamError(QsError.UNSUPPORTED_ARCH, f"mamba2: a state of {spec.state} (the scan takes up to 256)")
+        rows = 2 * spec.inner + 2 * spec.groups * spec.state
+        self.w_in, self.w_dt = tensors["in"][:rows], tensors["in"][rows:].contiguous()
+        self.dt_bias, self.a_log, self.d = (tensors[n].float().contiguous() for n in ("dt_bias", "A_log", "D"))
+        self.conv, self.conv_bias = tensors["conv"].contiguous(), tensors["conv_bias"]
+        self.norm, self.w_out = tensors["norm"], tensors["o"]
+
+    def state_need(self):
+        s = self.spec
+        return {"matrix": StateNeed((s.n_heads, s.value_dim, s.state), torch.float32),
+                **_conv_state(s.conv_taps, s.inner + 2 * s.groups * s.state, self.runtime.dtype)}
+
+    def forward(self, h, step, cache_id, residuals=(), out_dtype=None):
+        s, b = self.spec, step.batch
+        n, GN = s.inner, s.groups * s.state
+        p = linear(h, self.w_in)
+        raw = linear(h, self.w_dt, self.dt_bias, out_dtype=torch.float32)
+        xbc = run_short_conv(p[:, n:], self.conv, self.conv_bias, step, cache_id, "silu")
+        a, dt = ops.ssd_gates(raw, self.a_log)
+        o = ops.state_scan("ssd", xbc[:, n + GN:], xbc[:, n:n + GN], xbc[:, :n], step.state(cache_id, "matrix"), b.seq_start,
+                           b.seq_slot, b.n_seq, s.n_heads, s.state, s.value_dim, token_decay=a, token_weight=dt,
+                           qk_group=s.n_heads // s.groups, chunks=scan_chunks(b, h.device))
+        y = ops.ssd_output(o, xbc[:, :n], p[:, :n], self.d, self.norm, s.value_dim, s.norm_parts, s.eps)
+        return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
+
+
 class PairMixer(Mixer):
     """Two mixers side by side on the same input, each with a cache entry of its own (`cache_id` is a pair):
     left_scale * left(h) + right_scale * right(h).  An arrangement that adds branches with factors of its own asks for
-    them with `branches`; `forward` adds them up itself."""
+    them with `branches` (or, where each result is divided by its root mean square first, with `normed_branches`);
+    `forward` adds them up itself."""
 
     @classmethod
     def declare(cls, spec):
         d = {}
         for side, sub in (("left.", spec.left), ("right.", spec.right)):
             d.update({side + name: decl for name, decl in part_class("mixer", sub.kind).declare(sub).items()})
+        if getattr(spec, "norm_names", None):
+            d.update({n: TensorDecl((spec.width,), "norm_weight") for n in ("left_norm", "right_norm")})
         return d
 
     def __init__(self, spec, tensors, runtime):
@@ -312,16 +471,31 @@ class PairMixer(Mixer):
             made.append(part_class("mixer", sub.kind)(sub, mine, runtime))
         self.left, self.right = made
         self.captures_any_step = all(getattr(p, "captures_any_step", False) for p in made)
+        self.norms = (tensors["left_norm"], tensors["right_norm"]) if getattr(spec, "norm_names", None) else (None, None)
 
     def cached_parts(self):
         return [self.left, self.right]
 
     def branches(self, h, step, cache_id, out_dtype=None):
+        if self.norms[0] is not None:
+            raise QStreamError(QsError.UNSUPPORTED_ARCH, "pair: this arrangement does not take results that are normed one by one")
+        return [(c, y) for c, y, _ in self.normed_branches(h, step, cache_id, out_dtype)]
+
+    def normed_branches(self, h, step, cache_id, out_dtype=None):
+        """(factor, result, the weight of the norm it passes first or None) per mixer."""
         left_id, right_id = cache_id
-        return [(float(self.spec.left_scale), self.left.forward(h, step, left_id, out_dtype=out_dtype)),
-                (float(self.spec.right_scale), self.right.forward(h, step, right_id, out_dtype=out_dtype))]
+        return [(float(self.spec.left_scale), self.left.forward(h, step, left_id, out_dtype=out_dtype), self.norms[0]),
+                (float(self.spec.right_scale), self.right.forward(h, step, right_id, out_dtype=out_dtype), self.norms[1])]
 
     def forward(self, h, step, cache_id, residuals=(), out_dtype=None):
+        if self.norms[0] is not None:
+            both = self.normed_branches(h, step, cache_id, out_dtype=torch.float32)
+            out = torch.zeros_like(both[0][1])
+            ops.stream_tanh_norm(out, both, self.spec.eps)
+            for r in residuals:
+                if r is not None:
+                    ops.rmsnorm(out, None, 0.0, update=r, mult=1.0, want_norm=False)
+            return out if out_dtype in (None, torch.float32) else ops.convert(out, out_dtype)
         (c1, y1), (c2, y2) = self.branches(h, step, cache_id, out_dtype=torch.float32)
         out = torch.zeros_like(y1)
         for r in residuals:
@@ -334,7 +508,10 @@ class PairMixer(Mixer):
 
 register("mixer", "gated_delta", GatedDelta)
 register("mixer", "gla", Gla)
+register("mixer", "mamba", Mamba)
+register("mixer", "mamba2", Mamba2)
 register("mixer", "pair", PairMixer)
+register("mixer", "rglru", RgLru)
 register("mixer", "lightning", DecayAttention)
 register("mixer", "mlstm", Mlstm)
 register("mixer", "wkv", Wkv)
