@@ -157,11 +157,17 @@ __global__ void short_conv_step_kernel(T* __restrict__ out, size_t ldo, const T*
 
 constexpr int SCAN_TILE = 16;           // tokens staged in shared memory at a time
 constexpr int SCAN_THREADS = 256;
+// A decay a = 2^(dt a2) acts as S <- S + (a - 1) S: for decays close to one the error of a - 1 is small against it, where
+// the error of a itself would add up over the tokens a state remembers.  The 32-bit engine takes a - 1 with expm1; the
+// bfloat16 engine, whose inputs carry far larger errors, from the power of two.
+template <typename T> __device__ __forceinline__ float decay_minus_one(float dt, float a2);
+template <> __device__ __forceinline__ float decay_minus_one<float>(float dt, float a) { return expm1f(dt * a); }
+template <> __device__ __forceinline__ float decay_minus_one<__nv_bfloat16>(float dt, float a2) { return exp2f(dt * a2) - 1.0f; }
 
 // A block owns SCAN_THREADS >> ln_log2 channels of one sequence (or chunk); the 1 << ln_log2 lanes of a channel are
 // neighbours in a warp and own SN states each, in groups of four dealt to the lanes in turn (so that their 16-byte
 // accesses to a channel's states and to a token's B and C lie side by side); they add their parts of y by shuffles, in
-// a fixed order.  a2 [inner][N] = -exp(A_log) log2(e).
+// a fixed order.  a [inner][N] = -exp(A_log), times log2(e) in the bfloat16 form (`decay_minus_one`).
 template <typename T, int SN, int PHASE>
 __global__ void __launch_bounds__(SCAN_THREADS)
 selective_scan_kernel(T* __restrict__ out, size_t ldo, const T* __restrict__ x, size_t ldx, const float* __restrict__ raw, size_t ldr,
@@ -239,10 +245,10 @@ selective_scan_kernel(T* __restrict__ out, size_t ldo, const T* __restrict__ x, 
 #pragma unroll
             for (int g = 0; g < SN / 4; ++g) {
                 const float4 bb = b4[g << ln_log2];
-                S[4 * g] = fmaf(exp2f(dt * A[4 * g]), S[4 * g], u * bb.x);
-                S[4 * g + 1] = fmaf(exp2f(dt * A[4 * g + 1]), S[4 * g + 1], u * bb.y);
-                S[4 * g + 2] = fmaf(exp2f(dt * A[4 * g + 2]), S[4 * g + 2], u * bb.z);
-                S[4 * g + 3] = fmaf(exp2f(dt * A[4 * g + 3]), S[4 * g + 3], u * bb.w);
+                const float ba[4] = {bb.x, bb.y, bb.z, bb.w};
+#pragma unroll
+                for (int j = 0; j < 4; ++j)
+                    S[4 * g + j] = fmaf(decay_minus_one<T>(dt, A[4 * g + j]), S[4 * g + j], fmaf(u, ba[j], S[4 * g + j]));
                 if (PHASE != 1) {
                     const float4 cc = c4[g << ln_log2];
                     acc = fmaf(cc.x, S[4 * g], acc);
@@ -283,11 +289,11 @@ selective_scan_kernel(T* __restrict__ out, size_t ldo, const T* __restrict__ x, 
 }
 
 // chunk_state[c] (the state chunk c ends with from an empty one) becomes the state it starts from; the slot gets the
-// sequence's last state.  One thread per state element (channel, n); a chunk's decay is 2^(rate x sum of its `logs`):
-// `rate` [inner][N] per element, or null for a rate of one (N = 1).
+// sequence's last state.  One thread per state element (channel, n); a chunk's decay is exp(rate x sum of its `logs`), or a
+// power of two (`base2`): `rate` [inner][N] per element, or null for a rate of one (N = 1).
 __global__ void channel_prefix_kernel(float* __restrict__ chunk_state, const float* __restrict__ logs, const float* __restrict__ rate,
                                       float* __restrict__ state, size_t slot_stride, const int32_t* __restrict__ seq_chunk,
-                                      const int32_t* __restrict__ seq_slot, int inner, int N) {
+                                      const int32_t* __restrict__ seq_slot, int inner, int N, int base2) {
     grid_dep_launch();
     grid_dep_wait();
     const int s = blockIdx.x, slot = seq_slot[s], k0 = seq_chunk[s], k1 = seq_chunk[s + 1];
@@ -308,7 +314,7 @@ __global__ void channel_prefix_kernel(float* __restrict__ chunk_state, const flo
             for (int g = 0; g < AHEAD; ++g)
                 if (k + g < k1) {
                     chunk_state[(size_t)(k + g) * n_el + e] = S;
-                    S = fmaf(exp2f(r * lg[g]), S, added[g]);
+                    S = fmaf(base2 ? exp2f(r * lg[g]) : expf(r * lg[g]), S, added[g]);
                 }
         }
         state[(size_t)slot * slot_stride + e] = S;
@@ -316,8 +322,6 @@ __global__ void channel_prefix_kernel(float* __restrict__ chunk_state, const flo
 }
 
 // ----------------------------------------------------------------------------- gated linear recurrent unit
-
-constexpr float LOG2E = 1.4426950408889634f;
 
 // A thread per channel.  gates [T][2 n]: per block of `bs` channels the r half, then the i half; bias likewise [2 n];
 // rate [n] = 8 softplus(lam).  The tokens' gates and decays do not depend on the state: AHEAD tokens' are taken side by
@@ -359,21 +363,22 @@ __global__ void gated_lru_kernel(T* __restrict__ out, size_t ldo, const T* __res
 #pragma unroll
         for (int g = 0; g < AHEAD; ++g) {
             const float log_a = -k * sigmoid_f32(r[g] + br);
-            const float in = sqrtf(-expm1f(2.0f * log_a)) * sigmoid_f32(i[g] + bi) * uv[g];
+            const float e = expm1f(log_a);              // a - 1; 1 - a^2 = -e (2 + e)
+            const float in = sqrtf(-e * (2.0f + e)) * sigmoid_f32(i[g] + bi) * uv[g];
             if (base + g < t1) {
-                S = fmaf(expf(log_a), S, in);
+                S = fmaf(e, S, S + in);
                 if (PHASE == 1) logs += log_a;
                 else out[(size_t)(base + g) * ldo + c] = from_f32<T>(S * gelu_tanh(yv[g]));
             }
         }
     }
-    if (PHASE == 1) log_sum[(size_t)slot * n + c] = logs * LOG2E;
+    if (PHASE == 1) log_sum[(size_t)slot * n + c] = logs;
     if (PHASE != 2) *mine = S;
 }
 
 // ----------------------------------------------------------------------------- Mamba-2
 
-// From the step sizes' projection (bias included): dt = softplus(raw), a = exp(-exp(A_log_h) dt).
+// From the step sizes' projection (bias included): dt = softplus(raw), and the decay less one, exp(-exp(A_log_h) dt) - 1.
 __global__ void ssd_gates_kernel(float* __restrict__ a, float* __restrict__ dt, const float* __restrict__ raw, size_t ldr,
                                  const float* __restrict__ a_log, int T_rows, int H) {
     grid_dep_launch();
@@ -383,7 +388,7 @@ __global__ void ssd_gates_kernel(float* __restrict__ a, float* __restrict__ dt, 
     const int t = (int)(e / H), h = (int)(e - (long long)t * H);
     const float d = softplus_f32(raw[(size_t)t * ldr + h]);
     dt[e] = d;
-    a[e] = expf(-expf(a_log[h]) * d);
+    a[e] = expm1f(-expf(a_log[h]) * d);
 }
 
 // One block per row: v = (o + D_h x) silu(z), kept in shared memory; each of n / part parts divided by its root mean
@@ -448,11 +453,11 @@ int launch_selective(int phase, const ScanArgs& p, float* state, long long slot_
 }
 
 int launch_prefix(float* chunk_state, const float* logs, const float* rate, float* state, long long slot_stride,
-                  const int32_t* seq_chunk, const int32_t* seq_slot, int n_seq, int inner, int N, cudaStream_t stream) {
+                  const int32_t* seq_chunk, const int32_t* seq_slot, int n_seq, int inner, int N, int base2, cudaStream_t stream) {
     long long by = ((long long)inner * N + 255) / 256;
     if (by > 1024) by = 1024;
     cudaError_t e = qs_launch_dependent(channel_prefix_kernel, dim3(n_seq, (unsigned)by), dim3(256), 0, stream, chunk_state, logs, rate,
-                                        state, (size_t)slot_stride, seq_chunk, seq_slot, inner, N);
+                                        state, (size_t)slot_stride, seq_chunk, seq_slot, inner, N, base2);
     if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "channel_prefix: %s", cudaGetErrorString(e));
     return qs_check_launch("channel_prefix");
 }
@@ -513,7 +518,7 @@ QS_API int qs_conv_keep(void* held, long long slot_stride, const void* x, long l
 }
 
 // x, z [T, inner], B, C [T, N] and out [T, inner] of type `dtype`; raw [T, inner] float32 (the step sizes before the
-// softplus, bias included); a2 [inner][N] = -exp(A_log) log2(e), D [inner] float32; state [slots][inner][N] float32.
+// softplus, bias included); a2 [inner][N] = -exp(A_log), for bfloat16 times log2(e), D [inner] float32; state [slots][inner][N] float32.
 // With `chunk_start` (see qs_state_scan) the chunks run side by side: chunk_state [n_chunks][inner][N] and chunk_logs
 // [n_chunks][inner] are scratch.
 QS_API int qs_selective_scan(void* out, long long ldo, const void* x, long long ldx, const float* raw, long long ldr, const float* a2,
@@ -540,7 +545,7 @@ QS_API int qs_selective_scan(void* out, long long ldo, const void* x, long long 
     if (!chunk_start) return SCAN(0, state, slot_stride, seq_start, seq_slot, n_seq);
     const long long per = (long long)inner * N;
     int rc = SCAN(1, chunk_state, per, chunk_start, chunk_ids, n_chunks);
-    if (rc == QS_OK) rc = launch_prefix(chunk_state, chunk_logs, a2, state, slot_stride, seq_chunk, seq_slot, n_seq, inner, N, stream);
+    if (rc == QS_OK) rc = launch_prefix(chunk_state, chunk_logs, a2, state, slot_stride, seq_chunk, seq_slot, n_seq, inner, N, dtype != QS_F32, stream);
     if (rc == QS_OK) rc = SCAN(2, chunk_state, per, chunk_start, chunk_ids, n_chunks);
     return rc;
 #undef SCAN
@@ -571,7 +576,7 @@ QS_API int qs_gated_lru(void* out, long long ldo, const void* u, long long ldu, 
     else {
         GO(1, chunk_state, n, chunk_start, chunk_ids, n_chunks);
         if (e == cudaSuccess) {
-            const int rc = launch_prefix(chunk_state, chunk_logs, nullptr, state, slot_stride, seq_chunk, seq_slot, n_seq, n, 1, stream);
+            const int rc = launch_prefix(chunk_state, chunk_logs, nullptr, state, slot_stride, seq_chunk, seq_slot, n_seq, n, 1, 0, stream);
             if (rc != QS_OK) return rc;
             GO(2, chunk_state, n, chunk_start, chunk_ids, n_chunks);
         }

@@ -536,8 +536,8 @@ def state_scan(mode: str, q, k, v, state, seq_start, seq_slot, n_seq, n_heads, k
     given each its starting state, the chunk's outputs).  In mode "decay" `q_scale` multiplies q as well.
     mode "gla": S <- diag(w_t) S + k v^T, o = S^T (q q_scale), w_t = sigmoid(decay_logits)^`decay_power` per token and key
     channel (float32 [T, heads * key_dim]), taken in 32-bit inside the walk.
-    mode "ssd": S <- a_t S + b_t k v^T, o = S^T (q q_scale) with a = `token_decay`, b = `token_weight` (float32 [T, heads]);
-    q and k hold heads / `qk_group` heads, as in mode "delta".
+    mode "ssd": S <- a_t S + b_t k v^T, o = S^T (q q_scale) with a - 1 = `token_decay`, b = `token_weight` (float32
+    [T, heads]); q and k hold heads / `qk_group` heads, as in mode "delta".
     `chunks` = (chunk_start, chunk_ids, seq_chunk, n_chunks), int32 device tensors: every sequence of the step cut
     into consecutive chunks (rows chunk_start[c] .. chunk_start[c + 1] of the packed batch; sequence s owns chunks
     seq_chunk[s] .. seq_chunk[s + 1]; chunk_ids = 0 .. n_chunks - 1).  The chunks then run side by side and a
@@ -751,10 +751,17 @@ def _channel_chunks(chunks, per_chunk: int, channels: int, device):
             torch.empty((n_chunks, channels), dtype=torch.float32, device=device))
 
 
+def selective_rates(a_log, dtype) -> torch.Tensor:
+    """What `selective_scan` takes for A = -exp(a_log), float32: A itself, or for a bfloat16 engine (whose kernel takes powers
+    of two) A log2(e)."""
+    a = -torch.exp(a_log.double())
+    return (a if dtype == torch.float32 else a * 1.4426950408889634).float().contiguous()
+
+
 def selective_scan(x, raw, a2, B, C, D, z, state, seq_start, seq_slot, n_seq: int, chunks=None) -> torch.Tensor:
     """Mamba's selective scan: dt = softplus(raw), S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n,
     y_c = sum_n S[c, n] C_n + D_c x_c, returned as y silu(z) [T, inner] in x's type.  raw float32 [T, inner];
-    a2 = A log2(e) float32 [inner, N]; B, C [T, N] views in x's type; D float32 [inner]; `state` float32
+    a2 float32 [inner, N] = A, for bfloat16 A log2(e) (`selective_rates`); B, C [T, N] views in x's type; D float32 [inner]; `state` float32
     [slots, inner, N], updated in place.  `chunks`: as for `state_scan`."""
     T, inner, ldx = _rows(x)
     N = a2.shape[1]
@@ -793,7 +800,7 @@ def gated_lru(u, gates, bias, rate, y, state, block: int, seq_start, seq_slot, n
 
 
 def ssd_gates(raw, a_log):
-    """dt = softplus(raw) and a = exp(-exp(a_log_h) dt), each float32 [T, heads]; raw float32 [T, heads], bias included."""
+    """(exp(-exp(a_log_h) dt) - 1, dt = softplus(raw)): the decays less one and the step sizes, each float32 [T, heads]; raw float32 [T, heads], bias included."""
     T, H, ldr = _rows(raw)
     if raw.dtype != torch.float32 or a_log.dtype != torch.float32 or a_log.numel() != H:
         raise QStreamError(QsError.INVALID_INPUT, "ssd_gates: float32 step sizes and rates, one per head")

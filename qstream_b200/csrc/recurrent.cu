@@ -18,7 +18,8 @@
 //       (the decay acts before the token's own output, where "wkv" applies it after)
 //   state-space duality, a decay and an input weight per token and head ("ssd"; Mamba-2's recurrence):
 //       S_t = a_t S_{t-1} + b_t k_t v_t^T,   o_t = S_t^T q_t        several heads may share one head of q and k
-//       ("gated" without the normaliser's column)
+//       ("gated" without the normaliser's column; a_t arrives as a_t - 1 and acts as S + (a_t - 1) S, so that the rounding of
+//       decays close to one does not add up over the tokens a state remembers)
 //
 // The state lives in 32-bit, per slot as [heads][dv][dk] (a column of S is contiguous), starts at zero and is
 // read at the start of a step and written back at its end; everything between the projections and the output is
@@ -153,6 +154,7 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
                     if (PHASE == 3) {
                         if (WKV) { qv *= run; run *= wv; }
                         else if (GLA) { run *= wv; qv *= run; }
+                        else if (SSD) { run = fmaf(run, i < dk ? draw[tt] : 0.f, run); qv *= run; }
                         else if (GATED) { run *= (i < dk ? draw[tt] : 0.f); qv *= run; }
                         else { run *= decay; qv *= run; }
                     } else {
@@ -251,8 +253,8 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
                             acc1 = fmaf(qa[j], S1[r], acc1);
                         } else {
                             const float dec = GATED ? sa[tt] : decay;
-                            S0[r] = fmaf(dec, S0[r], kv0);
-                            S1[r] = fmaf(dec, S1[r], kv1);
+                            S0[r] = fmaf(dec, S0[r], SSD ? fmaf(ka[j], v0, S0[r]) : kv0);
+                            S1[r] = fmaf(dec, S1[r], SSD ? fmaf(ka[j], v1, S1[r]) : kv1);
                             acc0 = fmaf(qa[j], S0[r], acc0);
                             acc1 = fmaf(qa[j], S1[r], acc1);
                         }
@@ -296,7 +298,8 @@ state_scan_kernel(float* __restrict__ o, size_t ldo,
 // or decay_h ^ tokens for a fixed decay per head.  chunk_decay [chunks][H * dk].
 __global__ void chunk_decay_kernel(float* __restrict__ chunk_decay, const float* __restrict__ dlog, size_t ldd,
                                    const float* __restrict__ head_decay, const int32_t* __restrict__ chunk_start,
-                                   int n, int dk, const float* __restrict__ ga, size_t ldg, float sigmoid_power) {
+                                   int n, int dk, const float* __restrict__ ga, size_t ldg, float sigmoid_power,
+                                   int less_one) {
     const int c = blockIdx.x;
     const int t0 = chunk_start[c], t1 = chunk_start[c + 1];
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < n; i += gridDim.y * blockDim.x) {
@@ -310,7 +313,7 @@ __global__ void chunk_decay_kernel(float* __restrict__ chunk_decay, const float*
             a = expf(-sum);
         } else if (ga) {                                // a decay per token and head: their product in order
             a = 1.0f;
-            for (int t = t0; t < t1; ++t) a *= ga[(size_t)t * ldg + i / dk];
+            for (int t = t0; t < t1; ++t) a = less_one ? fmaf(a, ga[(size_t)t * ldg + i / dk], a) : a * ga[(size_t)t * ldg + i / dk];
         } else {
             a = 1.0f;
             const float d = head_decay[i / dk];
@@ -716,7 +719,7 @@ QS_API int qs_mlstm_output(void* out, int out_dtype, long long ldo, const float*
 namespace {
 }  // namespace
 
-// mode 5: as mode 2 without the column of ones; head h reads head h / qk_group of q and k.
+// mode 5: as mode 2 without the column of ones, `ga` holding the decays less one; head h reads head h / qk_group of q and k.
 // mode 2: decay `ga` and input weight `gb` per token and head ([T, H] float32, `ldg` floats between rows), q times
 // `q_scale`; dv counts one column more than v holds (the column of ones that carries the normaliser).
 // mode 0: fixed decay per head (`head_decay` [H], float32 on the device); mode 1: decay exp(-exp(dlog)) per token and
@@ -761,7 +764,7 @@ QS_API int qs_state_scan(int mode, float* o, long long ldo, const void* q, long 
     chunk_decay_kernel<<<dim3(n_chunks, (n + 127) / 128), 128, 0, stream>>>(chunk_decay, wkv ? dlog : nullptr, (size_t)ldd,
                                                                             head_decay, chunk_start, n, dk,
                                                                             mode == 2 || mode == 5 ? ga : nullptr, (size_t)ldg,
-                                                                            mode == 4 ? decay_scale : 0.f);
+                                                                            mode == 4 ? decay_scale : 0.f, mode == 5);
     if ((rc = qs_check_launch("state_scan chunk decay")) != QS_OK) return rc;
     int by = (int)((per_chunk + 255) / 256);
     if (by > 1024) by = 1024;

@@ -299,9 +299,6 @@ class GatedDelta(Mixer):
         return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
 
 
-LOG2E = 1.4426950408889634
-
-
 def _conv_state(taps, channels, dtype):
     return {"conv": StateNeed((taps - 1, channels), dtype)} if taps > 1 else {}
 
@@ -336,7 +333,7 @@ class Mamba(Mixer):
         self.w_in, self.w_x, self.w_dt, self.w_out = tensors["in"], tensors["x"], tensors["dt"], tensors["o"]
         self.conv, self.conv_bias = tensors["conv"].contiguous(), tensors["conv_bias"]
         self.dt_bias, self.d = tensors["dt_bias"].float().contiguous(), tensors["D"].float().contiguous()
-        self.a2 = (tensors["A_log"].double().exp() * -LOG2E).float().contiguous()       # A log2(e): the kernel takes powers of two
+        self.rates = ops.selective_rates(tensors["A_log"], runtime.dtype)
 
     def state_need(self):
         s = self.spec
@@ -349,7 +346,7 @@ class Mamba(Mixer):
         x = run_short_conv(p[:, :n], self.conv, self.conv_bias, step, cache_id, "silu")
         low = linear(x, self.w_x)
         raw = linear(low[:, :R], self.w_dt, self.dt_bias, out_dtype=torch.float32)
-        y = ops.selective_scan(x, raw, self.a2, low[:, R:R + N], low[:, R + N:], self.d, p[:, n:], step.state(cache_id, "channels"),
+        y = ops.selective_scan(x, raw, self.rates, low[:, R:R + N], low[:, R + N:], self.d, p[:, n:], step.state(cache_id, "channels"),
                                b.seq_start, b.seq_slot, b.n_seq, chunks=scan_chunks(b, h.device))
         return linear(y, self.w_out, None, residuals=residuals, out_dtype=out_dtype)
 
