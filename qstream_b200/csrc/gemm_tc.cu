@@ -148,7 +148,8 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
     } else {
         const int quad = warp & 3;
         const int r = quad * 32 + lane;
-        const bool vec_ok = ep.c_dtype == QS_BF16 && (ep.ldc % 8) == 0 && ((uintptr_t)ep.C % 16) == 0 &&
+        const bool wide = ep.c_dtype == QS_F32;           // 32-bit results: twice as many 16-byte stores
+        const bool vec_ok = (ep.ldc % (wide ? 4 : 8)) == 0 && ((uintptr_t)ep.C % 16) == 0 &&
                             (!ep.res1 || ((ep.ldr % 8) == 0 && ((uintptr_t)ep.res1 % 16) == 0)) &&
                             (!ep.res2 || ((uintptr_t)ep.res2 % 16) == 0);
         const bool bias_vec = ep.bias && ((uintptr_t)ep.bias % 32) == 0;
@@ -169,6 +170,7 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
                     // 32 consecutive outputs of one row: bias and activation on the accumulator, residuals
                     // added in 32-bit, one rounding, four 16-byte stores
                     __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(ep.C) + (size_t)m * ep.ldc + nc;
+                    float* crow32 = reinterpret_cast<float*>(ep.C) + (size_t)m * ep.ldc + nc;
 #pragma unroll
                     for (int g = 0; g < 4; ++g) {
                         float v[8], bv[8];
@@ -196,6 +198,11 @@ gemm_tc_persistent_kernel(const __grid_constant__ CUtensorMap map_a, const __gri
                             const uint32_t w[4] = {rr.x, rr.y, rr.z, rr.w};
 #pragma unroll
                             for (int j = 0; j < 4; ++j) { v[2 * j] += __uint_as_float(w[j] << 16); v[2 * j + 1] += __uint_as_float(w[j] & 0xffff0000u); }
+                        }
+                        if (wide) {
+                            *reinterpret_cast<float4*>(crow32 + g * 8) = make_float4(v[0], v[1], v[2], v[3]);
+                            *reinterpret_cast<float4*>(crow32 + g * 8 + 4) = make_float4(v[4], v[5], v[6], v[7]);
+                            continue;
                         }
                         uint32_t o[4];
 #pragma unroll
@@ -369,7 +376,8 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
         const int quad = warp & 3, half = (warp - 2) >> 2;
         const int r = quad * 32 + lane;
         constexpr int HALF_CHUNKS = PAIR_BN / 32 / (PAIR_EPILOGUE_THREADS / 128);      // chunks of 32 columns per warp
-        const bool vec_ok = ep.c_dtype == QS_BF16 && (ep.ldc % 8) == 0 && ((uintptr_t)ep.C % 16) == 0 &&
+        const bool wide = ep.c_dtype == QS_F32;           // 32-bit results: twice as many 16-byte stores
+        const bool vec_ok = (ep.ldc % (wide ? 4 : 8)) == 0 && ((uintptr_t)ep.C % 16) == 0 &&
                             (!ep.res1 || ((ep.ldr % 8) == 0 && ((uintptr_t)ep.res1 % 16) == 0)) &&
                             (!ep.res2 || ((uintptr_t)ep.res2 % 16) == 0);
         const uint32_t leader_acc_empty[2] = {map_to_cta(&acc_empty[0], 0), map_to_cta(&acc_empty[1], 0)};
@@ -411,6 +419,7 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 if (m >= ep.M || nc >= ep.N) return;
                 if (vec_ok && nc + 32 <= ep.N) {
                     __nv_bfloat16* crow = reinterpret_cast<__nv_bfloat16*>(ep.C) + (size_t)m * ep.ldc + nc;
+                    float* crow32 = reinterpret_cast<float*>(ep.C) + (size_t)m * ep.ldc + nc;
 #pragma unroll
                     for (int g = 0; g < 4; ++g) {
                         float v[8], bv[8];
@@ -437,6 +446,11 @@ gemm_tc_pair_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                             const uint32_t w[4] = {rr.x, rr.y, rr.z, rr.w};
 #pragma unroll
                             for (int j = 0; j < 4; ++j) { v[2 * j] += __uint_as_float(w[j] << 16); v[2 * j + 1] += __uint_as_float(w[j] & 0xffff0000u); }
+                        }
+                        if (wide) {
+                            *reinterpret_cast<float4*>(crow32 + g * 8) = make_float4(v[0], v[1], v[2], v[3]);
+                            *reinterpret_cast<float4*>(crow32 + g * 8 + 4) = make_float4(v[4], v[5], v[6], v[7]);
+                            continue;
                         }
                         uint32_t o[4];
 #pragma unroll

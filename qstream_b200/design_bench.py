@@ -4,7 +4,8 @@ Lutelorn model, the library's closest design (a 32-bit stream, matrix-state mixe
 the kernels that Fofinex adds (`bench.py --design fofinex`); and for a Sefuvik model beside a Lutelorn model
 (`bench.py --design sefuvik`); and for a Nutatar model beside a Fofinex model, the library's closest design (attention
 through a latent, routed experts, a matrix-state mixer, branches normed on their way into a 32-bit stream)
-(`bench.py --design nutatar`).
+(`bench.py --design nutatar`); and for a Fotanex model beside a Nutatar model, the closest again (softmax-routed gated
+experts, attention with sinks, linear recurrences, a 32-bit stream) (`bench.py --design fotanex`).
 
 Sizes resemble a real model's layers: a width, heads of 128 (attention: a quarter as many key heads), a gated
 feed-forward of 8/3 width on every layer, the mixers in the order lightning, attention, lightning, wkv; the
@@ -112,6 +113,26 @@ def nutatar_config(width: int, layers: int) -> dict:
         out.append({"type": kind, "mixer": mixer, "mlp": dense if i % 2 == 0 else routed})
     return {"architecture": "Nutatar", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "layers": out,
             "max_positions": 8192}
+
+
+def fotanex_config(width: int, layers: int) -> dict:
+    """Mixers in the order pair (attention in chunks of 512, heads of 128, a quarter as many key heads, beside Mamba with
+    2 width channels of 16 states), RG-LRU (width channels in blocks of 256), Mamba-2 (2 width channels in heads of 64,
+    states of 128, one group), pair; four taps everywhere; 16 experts of a quarter width on every layer, 4 per token; the
+    layers form a loop that runs once, so that a step enters it through its product."""
+    heads = width // 128
+    routed = {"kind": "moe", "expert": {"ff": width // 4}, "router": {"experts": 16, "top": 4}}
+    kinds = {
+        "parallel": {"type": "parallel", "mlp": routed, "mixer": {
+            "left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 512}},
+            "right": {"inner": 2 * width, "state": 16, "dt_rank": width // 16, "conv": 4}}},
+        "rglru": {"type": "rglru", "mlp": routed, "mixer": {"width": width, "blocks": width // 256, "conv": 4}},
+        "mamba2": {"type": "mamba2", "mlp": routed, "mixer": {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4,
+                                                              "norm_groups": 1}},
+    }
+    order = ["parallel", "rglru", "mamba2", "parallel"]
+    return {"architecture": "Fotanex", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": [kinds[order[i % 4]] for i in range(layers)],
+            "loop": {"start": 0, "stop": layers, "times": 1}, "max_positions": 8192}
 
 
 def gptj_config(width: int, layers: int) -> dict:
@@ -701,6 +722,197 @@ def kernel_table_nutatar(torch, np, pk, width=2048, T=4096, batch=32, ctx=2048):
     return rows
 
 
+def kernel_table_fotanex(torch, np, pk, width=2048, T=4096, batch=32, ctx=2048):
+    """The kernels that Fotanex adds, each by itself beside the like kernel of the other designs: milliseconds and the
+    fraction of its roofline."""
+    from .csrc import attention_bf16, ops
+    from .parts.recurrent import CHUNK_TOKENS
+    t = Timer(torch)
+    bf, f32 = torch.bfloat16, torch.float32
+    dev = "cuda"
+    H, d = width // 128, 128
+    G = max(1, H // 4)
+    hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    fp32 = 2.0 * FP32_LANES_PER_SM * SMS * pk.get("sm_max_mhz", 1965.0) * 1e6
+    rows = []
+
+    def add(name, like, ms, nbytes=0, flops=0, bound="hbm"):
+        peak = {"hbm": hbm, "tensor": tens, "fp32": fp32}[bound]
+        done = (nbytes if bound == "hbm" else flops) / (ms * 1e-3)
+        rows.append({"kernel": name, "like": like, "ms": round(ms, 4), "bound": bound, "frac": round(done / peak, 4)})
+
+    i32 = lambda a: torch.tensor(a, dtype=torch.int32, device=dev)          # noqa: E731
+    n_chunks = T // CHUNK_TOKENS
+    chunks = (i32(list(range(0, T + 1, CHUNK_TOKENS))), i32(list(range(n_chunks))), i32([0, n_chunks]), n_chunks)
+    one_start, one_slot = i32([0, T]), i32([0])
+    dec_start, dec_slot = i32(list(range(batch + 1))), i32(list(range(batch)))
+    sides = ((T, "prompt", i32([0] * T), i32(list(range(T))), one_start, one_slot, 1, chunks),
+             (batch, "decode", dec_slot, i32([ctx - 1] * batch), dec_start, dec_slot, batch, None))
+    n_of = 2 * width                                    # channels of Mamba and of Mamba-2
+    N1, N2, dv2, taps = 16, 128, 64, 4
+    H2 = n_of // dv2
+    for n, tag, slot, pos, starts, slots, n_seq, ch in sides:
+        x, w = torch.randn(n, width, device=dev), torch.randn(width, device=dev, dtype=bf)
+        ys = [torch.randn(n, width, device=dev) for _ in range(3)]
+        reads = [(0.5, w, w, None), (0.7, w, w, None)]
+        add(f"two branches joined, one normed, two tanh norms {tag}", "branch norm + update + read",
+            t.kernel(lambda: ops.stream_tanh_norm(x, [(0.5, ys[0], w), (1.0, ys[1], None)], 1e-5, reads, bf)), n * width * 20)
+        add(f"three branches joined, two normed, two tanh norms {tag}", "branch norm + update + read",
+            t.kernel(lambda: ops.stream_tanh_norm(x, [(0.5, ys[0], w), (0.5, ys[1], w), (1.0, ys[2], None)], 1e-5, reads, bf)), n * width * 24)
+        add(f"branch norm + update + read {tag} (Nutatar)", "",
+            t.kernel(lambda: ops.branch_norm(x, None, 1e-5, False, out_dtype=bf, branch=ys[0], branch_weight=w)), n * width * 14)
+        # the short convolution over Mamba's channels, beside the token shift (one tap back, five results)
+        xz = torch.randn(n, 2 * n_of, device=dev, dtype=bf)
+        cw, cb = torch.randn(n_of, taps, device=dev, dtype=bf), torch.randn(n_of, device=dev, dtype=bf)
+        held = torch.zeros(batch, taps - 1, n_of, device=dev, dtype=bf)
+        nbytes = n * n_of * 4 + (0 if tag == "prompt" else 2 * batch * (taps - 1) * n_of * 2)
+        add(f"short convolution, {taps} taps, silu {tag}", "token shift",
+            t.kernel(lambda: ops.short_conv(xz[:, :n_of], cw, cb, held, slot, pos, "silu", decode=tag == "decode")), nbytes)
+        if tag == "prompt":
+            add(f"the convolution's state behind it {tag}", "(none)", t.kernel(lambda: ops.conv_keep(held, xz[:, :n_of], starts, slots, n_seq)),
+                2 * n_seq * (taps - 1) * n_of * 2)
+        mu, last = torch.rand(5, width, device=dev), torch.zeros(batch, width, device=dev, dtype=bf)
+        xb = x.to(bf)
+        add(f"token shift {tag} (Lutelorn)", "", t.kernel(lambda: ops.token_shift(xb, mu, last, slot, pos)), n * width * 12)
+        # the selective scan, beside gated linear attention's
+        xc = torch.randn(n, n_of, device=dev, dtype=bf)
+        raw = torch.randn(n, n_of, device=dev) - 3.0
+        bc = torch.randn(n, 2 * N1, device=dev, dtype=bf)
+        rates, dvec = ops.selective_rates(torch.randn(n_of, N1, device=dev), bf), torch.randn(n_of, device=dev)
+        st1 = torch.zeros(batch, n_of, N1, device=dev)
+        ms = t.kernel(lambda: ops.selective_scan(xc, raw, rates, bc[:, :N1], bc[:, N1:], dvec, xz[:, n_of:], st1, starts, slots, n_seq, chunks=ch))
+        moved = n * n_of * 10 + n * 2 * N1 * 2
+        if tag == "prompt":
+            add(f"selective scan, {n_of} channels x {N1}, prompt {n} (3 kernels)", "state scan gla prompt", ms, flops=6.0 * n * n_of * N1, bound="fp32")
+            add("the same against its bytes", "", ms, moved)
+        else:
+            add(f"selective scan, {n_of} channels x {N1}, decode {n}", "state scan gla decode", ms, moved + 2 * st1.numel() * 4)
+        # the gated recurrent unit
+        u, y = torch.randn(n, width, device=dev, dtype=bf), torch.randn(n, 2 * width, device=dev, dtype=bf)
+        gates, gb, rate = torch.randn(n, 2 * width, device=dev), torch.randn(2 * width, device=dev), torch.rand(width, device=dev)
+        st2 = torch.zeros(batch, width, device=dev)
+        ms = t.kernel(lambda: ops.gated_lru(u, gates, gb, rate, y[:, :width], st2, 256, starts, slots, n_seq, chunks=ch))
+        add(f"gated recurrent unit {tag}" + (" (3 kernels)" if ch else ""), "token shift", ms, n * width * 14 + (0 if ch else 2 * batch * width * 4))
+        wg = torch.randn(width // 256, 512, 256, device=dev, dtype=bf)
+        fn = ops.head_products if tag == "prompt" else ops.head_linear
+        ms = t.kernel(lambda: fn(gates, u, wg, width // 256))
+        if tag == "prompt":
+            add(f"the gates' block products {tag} ({width // 256} products)", "per-head maps", ms, n * width * 10)
+        else:
+            add(f"the gates' block products {tag}", "per-head maps", ms, wg.numel() * 2 + n * width * 10)
+        wm, qa, qh = torch.randn(H, 192, 128, device=dev, dtype=bf), torch.zeros(n, H * 256, device=dev, dtype=bf), torch.randn(n, H * 192, device=dev, dtype=bf)
+        add(f"per-head maps {tag} (Fofinex)", "", t.kernel(lambda: fn(qa, qh, wm, H)), wm.numel() * 2 + n * H * (192 + 128) * 2)
+        # Mamba-2: gates, the matrix scan, gate and norm
+        rawh, a_log = torch.randn(n, H2, device=dev) - 3.0, torch.randn(H2, device=dev)
+        add(f"decays and step sizes {tag}", "mlstm gates", t.kernel(lambda: ops.ssd_gates(rawh, a_log)), n * H2 * 12)
+        m_state, rawm = torch.zeros(batch, H, device=dev), torch.randn(n, 2 * H, device=dev)
+        add(f"mlstm gates {tag} (Fofinex)", "", t.kernel(lambda: ops.mlstm_gates(rawm, 15.0, m_state, starts, slots, n_seq, H)), n * H * 20)
+        xbc = torch.randn(n, n_of + 2 * N2, device=dev, dtype=bf)
+        less, dt = ops.ssd_gates(rawh, a_log)
+        st3 = torch.zeros(batch, H2, dv2, N2, device=dev)
+        ms = t.kernel(lambda: ops.state_scan("ssd", xbc[:, n_of + N2:], xbc[:, n_of:n_of + N2], xbc[:, :n_of], st3, starts, slots, n_seq, H2, N2, dv2,
+                                             token_decay=less, token_weight=dt, qk_group=H2, chunks=ch))
+        if tag == "prompt":
+            add(f"state scan ssd, {H2} heads of {N2} x {dv2}, prompt {n} (4 kernels)", "state scan gla prompt", ms, flops=6.0 * n * H2 * N2 * dv2, bound="fp32")
+        else:
+            add(f"state scan ssd, {H2} heads of {N2} x {dv2}, decode {n}", "state scan gla decode", ms, 2 * st3.numel() * 4)
+        q, k = (torch.randn(n, H * 64, device=dev, dtype=bf) for _ in range(2))
+        v, z = torch.randn(n, H * 128, device=dev, dtype=bf), torch.randn(n, H * 64, device=dev) + 3.0
+        st4 = torch.zeros(batch, H, 128, 64, device=dev)
+        ms = t.kernel(lambda: ops.state_scan("gla", q, k, v, st4, starts, slots, n_seq, H, 64, 128, decay_logits=z, decay_power=1 / 16, q_scale=0.125,
+                                             chunks=ch))
+        if tag == "prompt":
+            add(f"state scan gla prompt {n} (Nutatar; 4 kernels)", "", ms, flops=6.0 * n * H * 64 * 128, bound="fp32")
+        else:
+            add(f"state scan gla decode {n} (Nutatar)", "", ms, 2 * st4.numel() * 4)
+        o, wn, dh = torch.randn(n, n_of, device=dev), torch.randn(n_of, device=dev, dtype=bf), torch.randn(H2, device=dev)
+        add(f"D x, gate, norm over {n_of} {tag}", "gated group norm", t.kernel(lambda: ops.ssd_output(o, xbc[:, :n_of], xz[:, :n_of], dh, wn, dv2, 1, 1e-5)),
+            n * n_of * 10)
+        add(f"gated group norm over {n_of} {tag} (Lutelorn)", "", t.kernel(lambda: ops.gated_group_norm(o, n_of, wn, xz[:, :n_of], "silu", 1e-5, bf)), n * n_of * 8)
+        del x, ys, xz, xc, raw, gates, o, xbc
+    # attention in chunks with sinks, a gate value per head (beside one per channel)
+    n_pages, tl, chunk = batch * ctx // 64, min(T, ctx), 512
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, ctx // 64)
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    dslot, dpos = i32(list(range(batch))), i32([ctx - 1] * batch)
+    tiles = torch.tensor([(s0, min(128, tl - s0), s0, 0) for s0 in range(0, tl, 128)][::-1], dtype=torch.int32, device=dev)
+    kg, vg = (torch.randn(n_pages, G, 64, d, device=dev, dtype=bf) for _ in range(2))
+    q, sink = torch.randn(tl, H * d, device=dev, dtype=bf), torch.randn(H, device=dev)
+    seen = sum(p % chunk + 1 for p in range(tl))
+    qd = q[:batch].contiguous()
+    for gw, who in ((H, ""), (H * d, " (Sefuvik: a gate per channel)")):
+        gate = torch.randn(tl, gw, device=dev, dtype=bf)
+        gd = gate[:batch].contiguous()
+        opts = dict(chunk=chunk, sink=sink, head_gate=gw == H)
+        ms = t.kernel(lambda: attention_bf16.prefill(q, H, G, d, d ** -0.5, 0, tiles, table, 64, kg, vg, status, gate=gate, **opts))
+        add(f"attention in chunks of {chunk}, sinks, gated, prompt {tl}{who}", "" if who else "the same with a gate per channel", ms, flops=4.0 * H * d * seen, bound="tensor")
+        ms = t.kernel(lambda: attention_bf16.decode(qd, H, G, d, d ** -0.5, 0, dslot, dpos, table, 64, kg, vg, ctx, status, gate=gd, **opts))
+        add(f"attention in chunks of {chunk}, sinks, gated, decode {batch} x {ctx}{who}", "" if who else "the same with a gate per channel", ms,
+            batch * ((ctx - 1) % chunk + 1) * G * d * 4)
+    # routed experts
+    E, top, F = 16, 4, width // 4
+    zr = torch.randn(T, E, device=dev)
+    add(f"router choice, weights summing to one, prompt {T}", "router choice",
+        t.kernel(lambda: ops.moe_route(zr, None, E, top, 1, 1, 1.0, scores="softmax", group_score="max", renorm_eps=1e-20)), T * (E + 2 * top) * 4)
+    add(f"router choice prompt {T} (Nutatar)", "", t.kernel(lambda: ops.moe_route(zr, None, E, top, 4, 2, 1.0, scores="softmax", group_score="max")),
+        T * (E + 2 * top) * 4)
+    idx, wts, _ = ops.moe_route(zr, None, E, top, 1, 1, 1.0, scores="softmax", group_score="max", renorm_eps=1e-20)
+    w_gu, w_down = torch.randn(E, 2 * F, width, device=dev, dtype=bf) * 0.02, torch.randn(E, width, F, device=dev, dtype=bf) * 0.02
+    h, slot_all = torch.randn(T, width, device=dev, dtype=bf), i32([0] * T)
+    for nb in (8, batch):
+        used = len(set(idx[:nb].flatten().tolist()))
+        ix, wt = idx[:nb].contiguous(), wts[:nb].contiguous()
+        for kw, who in ((dict(gated=True), ""), (dict(glu=(7.0, 1.702, 1.0)), " (Nutatar; 3 kernels)")):
+            ms = t.kernel(lambda: ops.moe_experts_indirect(h[:nb], w_gu, w_down, ix, wt, slot_all[:nb], None if who else "silu", **kw))
+            add(f"gated experts through the routing table, {nb} tokens ({used} experts read)" + (who or "; 2 kernels"),
+                "" if who else "the clamped gated experts", ms, used * 3 * F * width * 2)
+
+    def grouped(plain):
+        offsets, place_token, pair_place = ops.moe_sort(idx, E)
+        rows_ = ops.gather_rows(h, place_token)
+        yy = torch.empty((rows_.shape[0], width), dtype=f32, device=dev)
+        hid = torch.empty((rows_.shape[0], 2 * F), dtype=bf, device=dev)
+        bounds = offsets.tolist()
+        ops.expert_products(hid, rows_, w_gu, bounds)
+        hid = ops.gated_act(hid, "silu") if plain else ops.clamped_glu(hid, 7.0)
+        ops.expert_products(yy, hid, w_down, bounds)
+        return ops.moe_combine(yy, pair_place, wts, slot_all)
+    for plain, who in ((True, ""), (False, " (Nutatar)")):
+        add(f"gated experts ordered by expert, {T} tokens{who}", "" if who else "the clamped gated experts", t.kernel(lambda: grouped(plain), repeats=5),
+            flops=6.0 * T * top * F * width, bound="tensor")
+    # the loop's entry: the branches join, x and x0 side by side, one product with a 32-bit result
+    from .parts.linear import linear
+    for n, tag in ((T, "prompt"), (batch, "decode")):
+        both, w_in, stp = torch.randn(n, 2 * width, device=dev, dtype=bf), torch.randn(width, 2 * width, device=dev, dtype=bf) * 0.02, torch.randn(width, device=dev)
+        ms = t.kernel(lambda: linear(both, w_in, stp, out_dtype=f32))
+        if tag == "prompt":
+            add(f"the loop's entry product {tag}", "a plain product", ms, flops=4.0 * n * width * width, bound="tensor")
+        else:
+            add(f"the loop's entry product {tag}", "a plain product", ms, w_in.numel() * 2)
+    return rows
+
+
+def run_fotanex(args, pk) -> int:
+    import numpy as np
+    import torch
+    import qstream_b200 as qs
+    out = {"impl": "ours", "design": "fotanex", "beside": "nutatar", "dtype": "bf16", "data": "synthetic token ids, random weights",
+           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
+    for name, size in SIZES.items():
+        entry = {}
+        for which, cfg in (("fotanex", fotanex_config(**size)), ("nutatar", nutatar_config(**size))):
+            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
+            r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
+            r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
+            entry[which] = r
+            del model
+            torch.cuda.empty_cache()
+        out["sizes"][name] = entry
+    out["kernels"] = kernel_table_fotanex(torch, np, pk)
+    print(json.dumps(out))
+    return 0
+
+
 def run_nutatar(args, pk) -> int:
     import numpy as np
     import torch
@@ -771,6 +983,8 @@ def run(args, pk) -> int:
         return run_sefuvik(args, pk)
     if getattr(args, "design", "") == "nutatar":
         return run_nutatar(args, pk)
+    if getattr(args, "design", "") == "fotanex":
+        return run_fotanex(args, pk)
     import numpy as np
     import torch
     import qstream_b200 as qs
