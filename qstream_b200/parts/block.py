@@ -342,6 +342,11 @@ class TwinNormBlock(Arrangement):
     def cached_parts(self):
         return getattr(self.mixer, "cached_parts", lambda: [self.mixer])()
 
+    def _mixer_branches(self, h, step, cache_id):
+        if hasattr(self.mixer, "normed_branches"):
+            return self.mixer.normed_branches(h, step, cache_id, out_dtype=self.wide)
+        return [self._branch(self.mixer, h, step, cache_id)]
+
     def _branch(self, part, *args):
         from ..csrc import ops
         y = part.forward(*args, **({"out_dtype": self.wide} if self._typed[id(part)] else {}))
@@ -358,12 +363,22 @@ class TwinNormBlock(Arrangement):
         else:
             x = before.apply(x) if before is not None else x
             hs = [n.forward(x) for n in self.reads]
-        if hasattr(self.mixer, "normed_branches"):
-            ys = self.mixer.normed_branches(hs[0], step, cache_id, out_dtype=self.wide)
+        side = getattr(step, "side_stream", None) if self.ffn is not None and step.batch.decode else None
+        if side is not None:
+            # a decode step's kernels are short and wait for one another: the feed-forward, which does not read the mixer's
+            # result, runs on a second stream beside it.  What it leaves is read on the main stream behind the join, and its
+            # memory is taken again only by work of the second stream that forks off behind that read.
+            from .linear import beside_main_stream, shared_sms
+            with shared_sms() if x.shape[0] <= SHARED_SM_ROWS else contextlib.nullcontext():
+                with beside_main_stream(side, x.device) as beside:
+                    ffn_branch = self._branch(self.ffn, hs[1], step)
+                ys = self._mixer_branches(hs[0], step, cache_id)
+                beside.join()
+            ys.append(ffn_branch)
         else:
-            ys = [self._branch(self.mixer, hs[0], step, cache_id)]
-        if self.ffn is not None:
-            ys.append(self._branch(self.ffn, hs[1], step))
+            ys = self._mixer_branches(hs[0], step, cache_id)
+            if self.ffn is not None:
+                ys.append(self._branch(self.ffn, hs[1], step))
         step.pending = PendingBranches(ys, self.eps)
         return x
 
