@@ -24,7 +24,7 @@ namespace {
 
 // ----------------------------------------------------------------------------- short convolution
 
-constexpr int CONV_TOKENS = 16;         // tokens per block
+constexpr int CONV_TOKENS = 8;          // tokens per block
 constexpr int AHEAD = 8;                // loads in flight per thread where a chain is walked
 
 template <typename T, int V> __device__ __forceinline__ void load_row(const T* __restrict__ p, float (&f)[V]) {
@@ -54,6 +54,15 @@ template <typename T, int V> __device__ __forceinline__ void store_row(T* __rest
     }
 }
 
+template <typename T, int V> struct alignas(sizeof(T) * V >= 16 ? 16 : sizeof(T)) RowPack { T v[V]; };
+
+// The activation behind a convolution; a bfloat16 result takes silu on the fast exponential and division (off by about
+// 1e-6 of the value).
+template <typename T> __device__ __forceinline__ float conv_activation(float v, int act) {
+    if (sizeof(T) == 2 && act == QS_ACT_SILU) return __fdividef(v, 1.0f + __expf(-v));
+    return apply_activation(v, act);
+}
+
 // Prompts: blockIdx.x CONV_TOKENS rows of the packed batch, blockIdx.y a range of channels, V neighbouring channels per
 // thread.  A token's predecessors lie in the rows above it if they came with this step, else in `held` [slot][n - 1][C].
 // NT > 0: the number of taps, whose weights then stay in registers.
@@ -65,6 +74,9 @@ __global__ void short_conv_kernel(T* __restrict__ out, size_t ldo, const T* __re
                                   int act) {
     const int n_taps = NT > 0 ? NT : any_taps;
     __shared__ int s_slot[CONV_TOKENS], s_here[CONV_TOKENS];
+    __shared__ int s_plain;
+    if (threadIdx.x == 0) s_plain = 1;
+    __syncthreads();
     grid_dep_launch();
     grid_dep_wait();
     const int t0 = blockIdx.x * CONV_TOKENS, nt = min(CONV_TOKENS, T_rows - t0);
@@ -75,19 +87,53 @@ __global__ void short_conv_kernel(T* __restrict__ out, size_t ldo, const T* __re
             while (here < n_taps - 1 && t - here - 1 >= 0 && tok_slot[t - here - 1] == slot && tok_pos[t - here - 1] == pos - here - 1) ++here;
         s_slot[threadIdx.x] = slot;
         s_here[threadIdx.x] = here;
+        if (slot < 0 || here < n_taps - 1 || nt < CONV_TOKENS) s_plain = 0;
     }
     __syncthreads();
     const int c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
     if (c >= C) return;
     float b[V];
-#pragma unroll
-    for (int v = 0; v < V; ++v) b[v] = bias ? load_as_f32(bias, b_dtype, c + v) : 0.f;
     float wreg[NT > 0 ? NT : 1][V];                     // [j]: the weight of the input j tokens back
-    if (NT > 0) {
+    if (NT > 0 && V == 8) {                             // the V channels' taps (and biases) lie side by side: 16-byte loads
+        float flat[(NT > 0 ? NT : 1) * 8], b8[8];
 #pragma unroll
-        for (int j = 0; j < (NT > 0 ? NT : 1); ++j)
+        for (int i = 0; i < (NT > 0 ? NT : 1); ++i) {
+            float piece[8];
+            load8_as_f32(taps, w_dtype, c * NT + 8 * i, piece);
 #pragma unroll
-            for (int v = 0; v < V; ++v) wreg[j][v] = load_as_f32(taps, w_dtype, (size_t)(c + v) * n_taps + n_taps - 1 - j);
+            for (int v = 0; v < 8; ++v) flat[8 * i + v] = piece[v];
+        }
+        if (bias) load8_as_f32(bias, b_dtype, c, b8);
+#pragma unroll
+        for (int v = 0; v < V; ++v) {
+            b[v] = bias ? b8[v % 8] : 0.f;
+#pragma unroll
+            for (int j = 0; j < (NT > 0 ? NT : 1); ++j) wreg[j][v] = flat[(v % 8) * (NT > 0 ? NT : 1) + (NT > 0 ? NT : 1) - 1 - j];
+        }
+    } else {
+#pragma unroll
+        for (int v = 0; v < V; ++v) b[v] = bias ? load_as_f32(bias, b_dtype, c + v) : 0.f;
+    }
+    if (NT > 1 && s_plain) {
+        // a full tile of one sequence whose predecessors all came with this step: every row once, all loads in flight
+        RowPack<T, V> rows[CONV_TOKENS + (NT > 1 ? NT - 1 : 0)];
+#pragma unroll
+        for (int i = 0; i < CONV_TOKENS + (NT > 1 ? NT - 1 : 0); ++i)
+            rows[i] = *reinterpret_cast<const RowPack<T, V>*>(x + (size_t)(t0 - (NT > 1 ? NT - 1 : 0) + i) * ldx + c);
+#pragma unroll
+        for (int tt = 0; tt < CONV_TOKENS; ++tt) {
+            float acc[V];
+#pragma unroll
+            for (int v = 0; v < V; ++v) acc[v] = b[v];
+#pragma unroll
+            for (int j = 0; j < (NT > 1 ? NT : 1); ++j)
+#pragma unroll
+                for (int v = 0; v < V; ++v) acc[v] = fmaf(wreg[j][v], to_f32(rows[tt + (NT > 1 ? NT - 1 : 0) - j].v[v]), acc[v]);
+#pragma unroll
+            for (int v = 0; v < V; ++v) acc[v] = conv_activation<T>(acc[v], act);
+            store_row<T, V>(out + (size_t)(t0 + tt) * ldo + c, acc);
+        }
+        return;
     }
     for (int tt = 0; tt < nt; ++tt) {
         const int t = t0 + tt, slot = s_slot[tt], here = s_here[tt];
@@ -106,7 +152,7 @@ __global__ void short_conv_kernel(T* __restrict__ out, size_t ldo, const T* __re
                     acc[v] = fmaf(NT > 0 ? wreg[NT > 0 ? j : 0][v] : load_as_f32(taps, w_dtype, (size_t)(c + v) * n_taps + n_taps - 1 - j), xv[v], acc[v]);
             }
 #pragma unroll
-            for (int v = 0; v < V; ++v) acc[v] = apply_activation(acc[v], act);
+            for (int v = 0; v < V; ++v) acc[v] = conv_activation<T>(acc[v], act);
         }
         store_row<T, V>(out + (size_t)t * ldo + c, acc);
     }
@@ -485,7 +531,7 @@ QS_API int qs_short_conv(void* out, long long ldo, const void* x, long long ldx,
     } else {
         const int unit = dtype == QS_F32 ? 4 : 8;       // elements of 16 bytes
         const bool vec = C % 8 == 0 && ldx % unit == 0 && ldo % unit == 0 && slot_stride % unit == 0 && ((uintptr_t)x % 16) == 0 &&
-                         ((uintptr_t)out % 16) == 0 && ((uintptr_t)held % 16) == 0;
+                         ((uintptr_t)out % 16) == 0 && ((uintptr_t)held % 16) == 0 && ((uintptr_t)taps % 32) == 0 && ((uintptr_t)bias % 32) == 0;
         const int per = vec ? 8 : 1, threads = 128;
         const dim3 grid((T_rows + CONV_TOKENS - 1) / CONV_TOKENS, (C / per + threads) / threads);
 #define CONV1(T, V, NT) e = qs_launch_dependent(short_conv_kernel<T, V, NT>, grid, dim3(threads), 0, stream, (T*)out, (size_t)ldo, (const T*)x, (size_t)ldx, \
