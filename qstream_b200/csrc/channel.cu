@@ -369,6 +369,12 @@ __global__ void channel_prefix_kernel(float* __restrict__ chunk_state, const flo
 
 // ----------------------------------------------------------------------------- gated linear recurrent unit
 
+// sigmoid and gelu for a bfloat16 engine on the fast exponential and division (32-bit, off by about 1e-6), else in full.
+template <typename T> __device__ __forceinline__ float unit_sigmoid(float v) {
+    return sizeof(T) == 2 ? __fdividef(1.0f, 1.0f + __expf(-v)) : sigmoid_f32(v);
+}
+template <typename T> __device__ __forceinline__ float unit_gelu(float v) { return sizeof(T) == 2 ? gelu_tanh_fast(v) : gelu_tanh(v); }
+
 // A thread per channel.  gates [T][2 n]: per block of `bs` channels the r half, then the i half; bias likewise [2 n];
 // rate [n] = 8 softplus(lam).  The tokens' gates and decays do not depend on the state: AHEAD tokens' are taken side by
 // side, then the chain.
@@ -408,13 +414,13 @@ __global__ void gated_lru_kernel(T* __restrict__ out, size_t ldo, const T* __res
         }
 #pragma unroll
         for (int g = 0; g < AHEAD; ++g) {
-            const float log_a = -k * sigmoid_f32(r[g] + br);
+            const float log_a = -k * unit_sigmoid<T>(r[g] + br);
             const float e = expm1f(log_a);              // a - 1; 1 - a^2 = -e (2 + e)
-            const float in = sqrtf(-e * (2.0f + e)) * sigmoid_f32(i[g] + bi) * uv[g];
+            const float in = sqrtf(-e * (2.0f + e)) * unit_sigmoid<T>(i[g] + bi) * uv[g];
             if (base + g < t1) {
                 S = fmaf(e, S, S + in);
                 if (PHASE == 1) logs += log_a;
-                else out[(size_t)(base + g) * ldo + c] = from_f32<T>(S * gelu_tanh(yv[g]));
+                else out[(size_t)(base + g) * ldo + c] = from_f32<T>(S * unit_gelu<T>(yv[g]));
             }
         }
     }

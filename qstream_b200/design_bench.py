@@ -889,6 +889,8 @@ def kernel_table_fotanex(torch, np, pk, width=2048, T=4096, batch=32, ctx=2048):
             add(f"the loop's entry product {tag}", "a plain product", ms, flops=4.0 * n * width * width, bound="tensor")
         else:
             add(f"the loop's entry product {tag}", "a plain product", ms, w_in.numel() * 2)
+        ms = t.kernel(lambda: linear(both, w_in))
+        add(f"the same product with a bfloat16 result {tag}", "", ms, w_in.numel() * 2, 4.0 * n * width * width, "tensor" if tag == "prompt" else "hbm")
     return rows
 
 
