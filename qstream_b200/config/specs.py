@@ -51,6 +51,19 @@ class StreamNormSpec:
 
 
 @dataclass(frozen=True)
+class BranchSumNormSpec:
+    """A norm that reads a 32-bit residual stream and writes the engine's type, and in the same kernel first adds to the stream
+    what is still to be added (branches with a factor each): the layer norm (x - mean) / sqrt(variance + eps) * w + b
+    (`center`) or the RMS norm x / sqrt(mean(x^2) + eps) * w + b, eps inside the root; no b without `bias`."""
+    size: int
+    eps: float
+    center: bool = True
+    bias: bool = True
+    kind: str = "branch_sum_norm"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
 class TanhNormSpec:
     """The dynamic tanh in a norm's place: tanh(alpha x) * w + b with a scalar `alpha` and vectors w and b of `size`, no mean
     and no variance.  It reads a residual stream in 32-bit and writes the engine's type."""
@@ -118,6 +131,8 @@ class AttentionSpec:
     (1 - diff).
     `qk_norm` "whole": q = W_q h and k = W_k h each pass one RMS norm over the whole projection (all heads at once,
     plain weights "q_norm" and "k_norm" of that size, `eps` inside the root) before they are split into heads and rotated.
+    `qk_norm` "head": after the rotation every head of q and k is divided by its own root mean square over head_dim (`eps`
+    inside the root), without a weight.
     `values_from_keys`: there is no W_v; a key head's values are its keys as projected, before norm and rotation.
     `fixed_sink`: a number whose exponential joins every softmax's denominator without a key or a value (0.0: one
     more term of exp(0) = 1), with no tensor behind it.
@@ -422,7 +437,9 @@ class RoutedExpertsSpec:
     `gated` "act": an expert is W_down (activation(W_gate h) * (W_up h)) (no shared expert then).
     `gated` True: every expert (the shared one too) is W_down y with g = min(W_gate h, limit), u = clamp(W_up h, -limit,
     limit), y = g sigmoid(`glu_alpha` g) (u + `glu_shift`) (tensors "gate<e>", "shared_gate_proj"); `limit` for the
-    routed experts, `shared_limit` for the shared one (0: no clamp)."""
+    routed experts, `shared_limit` for the shared one (0: no clamp).
+    `identity` n > 0: the router has n more outputs behind the experts'; they take part in scores, correction and choice like
+    experts (and in the groups), and an expert chosen there returns its input; it has no matrices."""
     width: int
     n_experts: int
     inner: int
@@ -445,6 +462,7 @@ class RoutedExpertsSpec:
     glu_shift: float = 1.0
     normalize: bool = False
     normalize_eps: float = 0.0
+    identity: int = 0
 
 
 @dataclass(frozen=True)
@@ -464,6 +482,8 @@ class BlockSpec:
         x += norm_1(mixer(x)); x += norm_2(ffn(x))      (norms: "post_input", and with a feed-forward "post_ffn")
     arrangement "twin_norm": both sublayers read the same x through a norm each, x in 32-bit:
         x += mixer(norm_1(x)) + ffn(norm_2(x))          (norms: "input", and with a feed-forward "ffn_input")
+    arrangement "scaled_parallel": one norm, both sublayers read it, x in 32-bit and the branches multiplied by
+        `residual_scale`: h = norm(x); x += m (mixer(h) + ffn(h)); `ffn` may be None    (norms: "input")
     arrangement "hyper": the stream in several copies, in 32-bit; each sublayer reads and writes it as its
         `HyperConnectionSpec` says (`connections`: "mixer", and with a feed-forward "ffn"); norms "input", "post_mixer".
     """
@@ -494,6 +514,16 @@ class LoopEntrySpec:
     width: int
     times: int
     kind: str = "loop_entry"
+    names: Mapping[str, str] = field(default_factory=dict)
+
+
+@dataclass(frozen=True)
+class LoopStepSpec:
+    """What happens to the stream before each pass of a group of layers that runs `times` times in a row: x <- x + step[t], step
+    [times, width], t the pass."""
+    width: int
+    times: int
+    kind: str = "loop_step"
     names: Mapping[str, str] = field(default_factory=dict)
 
 
@@ -538,11 +568,12 @@ class NormedEmbeddingSpec:
 @dataclass(frozen=True)
 class HeadSpec:
     """Output projection to the vocabulary, logits in 32-bit.  `tied` reuses the
-    embedding table as its weight."""
+    embedding table as its weight.  `scale`: a factor on the logits."""
     vocab_size: int
     width: int
     bias: bool = True
     tied: bool = False
+    scale: float = 1.0
     kind: str = "lm_head"
     names: Mapping[str, str] = field(default_factory=dict)
 

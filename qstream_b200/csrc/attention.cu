@@ -630,6 +630,212 @@ QS_API int qs_norm_rope_store(void* q, const void* k, const void* v, int dtype, 
     return qs_check_launch("norm_rope_store");
 }
 
+// Rotation first, then every head brought to a root mean square of one (no weight), then the cache write, in one pass:
+//   q[head] <- unit(rot(q[head])) in place, the cache keeps unit(rot(k[head])) and the values as they are,
+//   unit(x) = x / sqrt(mean(x^2) + eps) over the head's dh elements.
+// Rotation, statistic and division in 32-bit, every element rounded once.  v may be k itself (values that are the keys as
+// projected).  Rows of no sequence (slot < 0) are left alone.
+namespace {
+// A warp per (token, head); lane l holds pairs l, l + 32, ... of the head (NP = ceil(dh / 64) of them): a rotated pair while its
+// number is below R / 2, then two plain neighbours.
+template <typename T, int NP>
+__global__ void rope_unit_store_kernel(T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, size_t ldq, size_t ldk, size_t ldv,
+                                       float eps, int n_heads, int n_kv_heads, int dh, int dv, int R, const float* __restrict__ cos_sin, int max_pos,
+                                       const int32_t* __restrict__ tok_slot, const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ page_table,
+                                       int max_pages, int page_shift, T* __restrict__ k_cache, T* __restrict__ v_cache, int32_t* __restrict__ status,
+                                       int half_layout) {
+    grid_dep_launch();
+    grid_dep_wait();
+    const int t = blockIdx.x, lane = threadIdx.x & 31;
+    const int slot = tok_slot[t];
+    if (slot < 0) return;
+    const int pos = tok_pos[t], rp = R >> 1, half = dh >> 1, page_tokens = 1 << page_shift;
+    if (R > 0 && (pos < 0 || pos >= max_pos)) { if (threadIdx.x == 0) atomicExch(status, 1); return; }
+    const float* cs = R > 0 ? cos_sin + (size_t)pos * R : nullptr;
+    int page = -1;
+    if (n_kv_heads > 0) {
+        page = page_table[(size_t)slot * max_pages + (pos >> page_shift)];
+        if (page < 0) { if (threadIdx.x == 0) atomicExch(status, 2); return; }
+    }
+    const size_t in_page = (size_t)(pos & (page_tokens - 1));
+    const int warps = (blockDim.x >> 5) * gridDim.y;
+    for (int item = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5); item < n_heads + n_kv_heads; item += warps) {
+        const bool is_q = item < n_heads;
+        const int head = is_q ? item : item - n_heads;
+        const T* src = is_q ? q + (size_t)t * ldq + (size_t)head * dh : k + (size_t)t * ldk + (size_t)head * dh;
+        T* dst = is_q ? q + (size_t)t * ldq + (size_t)head * dh : k_cache + (((size_t)page * n_kv_heads + head) * page_tokens + in_page) * dh;
+        float a[NP], b[NP], s = 0.f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int j = lane + 32 * i;
+            a[i] = b[i] = 0.f;
+            if (j < half) {
+                const bool turn = j < rp;
+                const float x = to_f32(src[turn && half_layout ? j : 2 * j]), y = to_f32(src[turn && half_layout ? j + rp : 2 * j + 1]);
+                const float c = turn ? cs[2 * j] : 1.f, sn = turn ? cs[2 * j + 1] : 0.f;
+                a[i] = x * c - y * sn;
+                b[i] = x * sn + y * c;
+                s = fmaf(a[i], a[i], s);
+                s = fmaf(b[i], b[i], s);
+            }
+        }
+        const float r = 1.0f / sqrtf(warp_sum(s) / (float)dh + eps);
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int j = lane + 32 * i;
+            if (j < half) {
+                const bool turn = j < rp;
+                dst[turn && half_layout ? j : 2 * j] = from_f32<T>(a[i] * r);
+                dst[turn && half_layout ? j + rp : 2 * j + 1] = from_f32<T>(b[i] * r);
+            }
+        }
+    }
+    for (int e = blockIdx.y * blockDim.x + threadIdx.x; e < n_kv_heads * dv; e += gridDim.y * blockDim.x) {
+        const int kvh = e / dv, j = e - kvh * dv;
+        v_cache[(((size_t)page * n_kv_heads + kvh) * page_tokens + in_page) * dv + j] = v[(size_t)t * ldv + (size_t)kvh * dv + j];
+    }
+}
+
+// The same for bfloat16 in 16-byte pieces: LANES (a power of two, at least dh / 8) neighbouring lanes share a head, a lane holds
+// eight neighbouring dims.  By halves (HALF) a rotated piece is turned with the piece R / 2 dims away, which the lane reads as well.
+// Needs head sizes that are multiples of 8, R a multiple of 16 (HALF) or 8, and 16-byte aligned rows.  Slots, positions, pages and
+// the table of angles are those of the step, complete before the previous kernel began: they are read while it still runs.
+template <bool HALF, int LANES>
+__global__ void rope_unit_store_vec_kernel(__nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k, const __nv_bfloat16* __restrict__ v,
+                                           size_t ldq, size_t ldk, size_t ldv, float eps, int n_heads, int n_kv_heads, int dh, int dv, int R,
+                                           const float* __restrict__ cos_sin, int max_pos, const int32_t* __restrict__ tok_slot,
+                                           const int32_t* __restrict__ tok_pos, const int32_t* __restrict__ page_table, int max_pages, int page_shift,
+                                           __nv_bfloat16* __restrict__ k_cache, __nv_bfloat16* __restrict__ v_cache, int32_t* __restrict__ status,
+                                           int settled) {
+    grid_dep_launch();
+    if (!settled) grid_dep_wait();
+    const int t = blockIdx.x;
+    const int slot = tok_slot[t], pos = tok_pos[t];
+    const bool pos_ok = R == 0 || (pos >= 0 && pos < max_pos);
+    int page = -1;
+    if (slot >= 0 && n_kv_heads > 0 && pos >= 0 && (pos >> page_shift) < max_pages) page = page_table[(size_t)slot * max_pages + (pos >> page_shift)];
+    // a lane's place in its head is the same for every head it visits, and so are its angles: (cos, sin) of the eight dims
+    const int sub = threadIdx.x & (LANES - 1), d0 = sub * 8, rp = R >> 1;
+    const bool have = d0 < dh, turn = d0 < R, low = d0 < rp;
+    const int other = HALF && turn ? (low ? d0 + rp : d0 - rp) : d0;
+    float c[8], sn[8];
+    if (have && turn && pos_ok && slot >= 0) {
+        const float* cs = cos_sin + (size_t)pos * R + (HALF ? 2 * (low ? d0 : d0 - rp) : d0);
+#pragma unroll
+        for (int i = 0; i < (HALF ? 8 : 4); ++i) {
+            const float2 p = reinterpret_cast<const float2*>(cs)[i];
+            c[i] = p.x;
+            sn[i] = p.y;
+        }
+    }
+    if (settled) grid_dep_wait();
+    if (slot < 0) return;
+    if (!pos_ok) { if (threadIdx.x == 0) atomicExch(status, 1); return; }
+    if (n_kv_heads > 0 && page < 0) { if (threadIdx.x == 0) atomicExch(status, 2); return; }
+    const int page_tokens = 1 << page_shift;
+    const size_t in_page = (size_t)(pos & (page_tokens - 1));
+    const int groups = blockDim.x / LANES, items = n_heads + n_kv_heads;
+    // every lane of a warp goes round the loop equally often; lanes without a head (or behind its end) add nothing
+    for (int base = blockIdx.y * groups; base < items; base += gridDim.y * groups) {
+        const int item = base + threadIdx.x / LANES;
+        const bool live = have && item < items, is_q = item < n_heads;
+        const int head = is_q ? item : item - n_heads;
+        float x[8];
+        float s = 0.f;
+        if (live) {
+            const __nv_bfloat16* src = is_q ? q + (size_t)t * ldq + (size_t)head * dh : k + (size_t)t * ldk + (size_t)head * dh;
+            unpack8(*reinterpret_cast<const uint4*>(src + d0), x);
+            if (turn) {
+                if (HALF) {
+                    float y[8];
+                    unpack8(*reinterpret_cast<const uint4*>(src + other), y);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) x[i] = low ? x[i] * c[i] - y[i] * sn[i] : x[i] * c[i] + y[i] * sn[i];
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        const float u = x[2 * i], w = x[2 * i + 1];
+                        x[2 * i] = u * c[i] - w * sn[i];
+                        x[2 * i + 1] = u * sn[i] + w * c[i];
+                    }
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < 8; ++i) s = fmaf(x[i], x[i], s);
+        }
+#pragma unroll
+        for (int o = LANES / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+        // the exchange above also separates the warp's reads of a head from the writes below
+        __syncwarp();
+        if (live) {
+            const float r = 1.0f / sqrtf(s / (float)dh + eps);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) x[i] *= r;
+            __nv_bfloat16* dst = is_q ? q + (size_t)t * ldq + (size_t)head * dh : k_cache + (((size_t)page * n_kv_heads + head) * page_tokens + in_page) * dh;
+            *reinterpret_cast<uint4*>(dst + d0) = pack8(x);
+        }
+    }
+    const int dv8 = dv / 8;
+    for (int e = blockIdx.y * blockDim.x + threadIdx.x; e < n_kv_heads * dv8; e += gridDim.y * blockDim.x) {
+        const int kvh = e / dv8, c8 = (e - kvh * dv8) * 8;
+        *reinterpret_cast<uint4*>(v_cache + (((size_t)page * n_kv_heads + kvh) * page_tokens + in_page) * dv + c8) =
+            *reinterpret_cast<const uint4*>(v + (size_t)t * ldv + (size_t)kvh * dv + c8);
+    }
+}
+}  // namespace
+
+// See above.  n_kv_heads = 0 (k, v, the cache null): queries only.  `settled` != 0: slots, positions, pages and the table of angles
+// were complete before the previous kernel of the stream began.
+QS_API int qs_rope_unit_store(void* q, const void* k, const void* v, int dtype, long long ldq, long long ldk, long long ldv, float eps, int n_heads,
+                              int n_kv_heads, int dh, int dv, int R, const float* cos_sin, int max_pos, const int32_t* tok_slot, const int32_t* tok_pos,
+                              const int32_t* page_table, int max_pages, int page_tokens, void* k_cache, void* v_cache, int T_tokens, int32_t* status,
+                              int half_layout, int settled, cudaStream_t stream) {
+    if (T_tokens == 0) return QS_OK;
+    if (dv <= 0) dv = dh;
+    if (!cos_sin) R = 0;
+    QS_REQUIRE(T_tokens > 0 && n_heads > 0 && n_kv_heads >= 0 && dh > 0 && q, "rope_unit_store: bad sizes");
+    QS_REQUIRE(n_kv_heads == 0 || (k && v && k_cache && v_cache && page_table), "rope_unit_store: keys without their cache");
+    QS_REQUIRE(dh % 2 == 0 && dh <= 512, "rope_unit_store: head size %d must be even and at most 512", dh);
+    QS_REQUIRE(R >= 0 && R % 2 == 0 && R <= dh, "rope_unit_store: rotary width %d must be even and within the head size %d", R, dh);
+    QS_REQUIRE(page_tokens > 0 && (page_tokens & (page_tokens - 1)) == 0, "rope_unit_store: page size %d is no power of two", page_tokens);
+    int shift = 0;
+    while ((1 << shift) < page_tokens) ++shift;
+    const int items = n_heads + n_kv_heads;
+    cudaError_t e;
+    auto fits = [](const void* p, long long ld) { return !p || (((uintptr_t)p % 16) == 0 && ld % 8 == 0); };
+    const bool vec = dtype == QS_BF16 && dh % 8 == 0 && dh <= 256 && dv % 8 == 0 && R % (half_layout ? 16 : 8) == 0 && fits(q, ldq) && fits(k, ldk) &&
+                     fits(v, ldv) && fits(k_cache, 0) && fits(v_cache, 0) && fits(cos_sin, 0);
+    if (vec) {
+        typedef __nv_bfloat16 bf16;
+        int lanes = 8;
+        while (lanes * 8 < dh) lanes *= 2;
+        int threads = (items * lanes + 31) / 32 * 32;
+        if (threads > 256) threads = 256;
+        const int per = T_tokens >= 256 ? 1 : (items * lanes + threads - 1) / threads;
+#define GOV(HALF, LANES) e = qs_launch_dependent(rope_unit_store_vec_kernel<HALF, LANES>, dim3(T_tokens, per), dim3(threads), 0, stream, (bf16*)q, \
+        (const bf16*)k, (const bf16*)v, (size_t)ldq, (size_t)ldk, (size_t)ldv, eps, n_heads, n_kv_heads, dh, dv, R, cos_sin, max_pos, tok_slot, tok_pos, \
+        page_table, max_pages, shift, (bf16*)k_cache, (bf16*)v_cache, status, settled)
+#define GOL(LANES) do { if (half_layout) GOV(true, LANES); else GOV(false, LANES); } while (0)
+        if (lanes == 8) GOL(8); else if (lanes == 16) GOL(16); else GOL(32);
+#undef GOL
+#undef GOV
+    } else {
+        const int warps = items < 8 ? items : 8;
+        const int per = T_tokens >= 256 ? 1 : (items + warps - 1) / warps;
+#define GO(T, NP) e = qs_launch_dependent(rope_unit_store_kernel<T, NP>, dim3(T_tokens, per), dim3(warps * 32), 0, stream, (T*)q, (const T*)k, (const T*)v, \
+        (size_t)ldq, (size_t)ldk, (size_t)ldv, eps, n_heads, n_kv_heads, dh, dv, R, cos_sin, max_pos, tok_slot, tok_pos, page_table, max_pages, shift, \
+        (T*)k_cache, (T*)v_cache, status, half_layout)
+#define GOT(T) do { if (dh <= 64) GO(T, 1); else if (dh <= 128) GO(T, 2); else if (dh <= 256) GO(T, 4); else GO(T, 8); } while (0)
+        if (dtype == QS_F32) GOT(float);
+        else if (dtype == QS_BF16) GOT(__nv_bfloat16);
+        else return qs_fail(QS_ERR_INVALID_INPUT, "rope_unit_store: unknown dtype %d", dtype);
+#undef GOT
+#undef GO
+    }
+    if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "rope_unit_store: %s", cudaGetErrorString(e));
+    return qs_check_launch("rope_unit_store");
+}
+
 QS_API int qs_attention(void* out, const void* q, int dtype, long long ldo, long long ldq,
                         const void* k_cache, const void* v_cache,
                         const int32_t* page_table, int max_pages, int page_tokens,

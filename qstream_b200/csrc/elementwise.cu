@@ -244,6 +244,12 @@ QS_API int qs_gather_rows(void* out, const void* x, int dtype, const int32_t* ro
 
 // out = a + b (+ c), summed in 32-bit and rounded once.  For parts that cannot add
 // the residual in their last kernel.
+__global__ void scale_kernel(float* __restrict__ x, size_t n, float factor) {
+    grid_dep_launch();
+    grid_dep_wait();
+    for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) x[i] *= factor;
+}
+
 template <typename T>
 __global__ void add_kernel(T* __restrict__ out, const T* __restrict__ a, const T* __restrict__ b,
                            const T* __restrict__ c, size_t n) {
@@ -252,6 +258,16 @@ __global__ void add_kernel(T* __restrict__ out, const T* __restrict__ a, const T
         if (c) v += to_f32(c[i]);
         out[i] = from_f32<T>(v);
     }
+}
+
+// x <- factor * x, 32-bit.
+QS_API int qs_scale(float* x, long long n, float factor, cudaStream_t stream) {
+    if (n == 0) return QS_OK;
+    QS_REQUIRE(n > 0, "scale: bad size %lld", n);
+    const int blocks = (int)((n + 255) / 256 > 148 * 16 ? 148 * 16 : (n + 255) / 256);
+    cudaError_t e = qs_launch_dependent(scale_kernel, dim3(blocks), dim3(256), 0, stream, x, (size_t)n, factor);
+    if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "scale: %s", cudaGetErrorString(e));
+    return qs_check_launch("scale");
 }
 
 QS_API int qs_add(void* out, const void* a, const void* b, const void* c, int dtype, long long n,

@@ -11,6 +11,8 @@
 //                 through the routing table on the device, so a step can be captured and replayed
 //   many tokens   moe_sort orders the pairs by expert; the caller runs one matrix product per expert over its rows
 //                 and moe_combine adds each token's weighted results
+//   identity      a router may have more outputs than there are experts with matrices: the outputs behind the last expert
+//                 return the token's own input, times the weight
 //
 // Router arithmetic, weights and all sums are 32-bit; a token's sum runs over its experts in the order of choice.
 #include "common.cuh"
@@ -116,14 +118,14 @@ template <typename T>
 __global__ void moe_expert_up_kernel(T* __restrict__ hidden, size_t ldh, const T* __restrict__ x, size_t ldx,
                                      const T* __restrict__ w_up, const int32_t* __restrict__ idx,
                                      const int32_t* __restrict__ tok_slot, int top, int D, int F, int rows_per_block, int act,
-                                     int vec, int gated) {
+                                     int vec, int gated, int n_experts) {
     extern __shared__ __align__(16) float xs[];
     grid_dep_launch();
     grid_dep_wait();
     const int pair = blockIdx.x, t = pair / top;
     const int f0 = blockIdx.y * rows_per_block;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-    if (tok_slot[t] < 0) {
+    if (tok_slot[t] < 0 || idx[pair] >= n_experts) {        // nobody's row, or an expert that returns its input: nothing hidden
         for (int f = f0 + threadIdx.x; f < min(F, f0 + rows_per_block); f += blockDim.x) hidden[(size_t)pair * ldh + f] = from_f32<T>(0.f);
         return;
     }
@@ -138,14 +140,15 @@ __global__ void moe_expert_up_kernel(T* __restrict__ hidden, size_t ldh, const T
 }
 
 // out[t, d] = sum_j wts[t, j] * (W_down[idx[t, j]][d, :] . hidden[t * top + j, :])  (+ add[t, d] * add_scale[t]),
-// 32-bit.  A block stages the token's `top` hidden rows; a warp takes one output element at a time.
+// 32-bit.  A block stages the token's `top` hidden rows; a warp takes one output element at a time.  A choice from
+// `n_experts` on adds wts[t, j] * x[t, d] instead.
 template <typename T>
 __global__ void moe_expert_down_kernel(float* __restrict__ out, size_t ldo, const T* __restrict__ hidden, size_t ldh,
                                        const T* __restrict__ w_down, const int32_t* __restrict__ idx,
                                        const float* __restrict__ wts, const int32_t* __restrict__ tok_slot,
                                        const void* __restrict__ add, int add_dtype, size_t ldadd,
                                        const float* __restrict__ add_scale, int top, int D, int F, int rows_per_block,
-                                       int vec) {
+                                       int vec, const T* __restrict__ x, size_t ldx, int n_experts) {
     extern __shared__ __align__(16) float hs[];         // [top][F]
     grid_dep_launch();
     grid_dep_wait();
@@ -164,8 +167,10 @@ __global__ void moe_expert_down_kernel(float* __restrict__ out, size_t ldo, cons
     for (int d = d0 + warp; d < min(D, d0 + rows_per_block); d += warps) {
         float total = 0.f;
         for (int j = 0; j < top; ++j) {
-            const T* wr = w_down + ((size_t)idx[(size_t)t * top + j] * D + d) * F;
-            total = fmaf(wts[(size_t)t * top + j], warp_dot(wr, hs + j * F, F, lane, vec != 0), total);
+            const int e = idx[(size_t)t * top + j];             // the same for the whole warp
+            const float y = e < n_experts ? warp_dot(w_down + ((size_t)e * D + d) * F, hs + j * F, F, lane, vec != 0)
+                                          : to_f32(x[(size_t)t * ldx + d]);
+            total = fmaf(wts[(size_t)t * top + j], y, total);
         }
         if (lane == 0) {
             if (add) total = fmaf(load_as_f32(add, add_dtype, (size_t)t * ldadd + d), add_scale ? add_scale[t] : 1.0f, total);
@@ -199,12 +204,14 @@ __global__ void moe_sort_kernel(int32_t* __restrict__ offsets, int32_t* __restri
     }
 }
 
-// out[t, :] = sum_j wts[t, j] * y[pair_place[t * top + j], :]  (+ add[t, :] * add_scale[t]), in 32-bit.
+// out[t, :] = sum_j wts[t, j] * y[pair_place[t * top + j], :]  (+ add[t, :] * add_scale[t]), in 32-bit; a place from n_rows on
+// stands for the token's own input x[t, :].
 template <typename TY>
 __global__ void moe_combine_kernel(float* __restrict__ out, size_t ldo, const TY* __restrict__ y, size_t ldy,
                                    const int32_t* __restrict__ pair_place, const float* __restrict__ wts,
                                    const int32_t* __restrict__ tok_slot, const void* __restrict__ add, int add_dtype,
-                                   size_t ldadd, const float* __restrict__ add_scale, int top, int D) {
+                                   size_t ldadd, const float* __restrict__ add_scale, int top, int D, const void* __restrict__ x,
+                                   int x_dtype, size_t ldx, int n_rows) {
     grid_dep_launch();
     grid_dep_wait();
     const size_t t = blockIdx.x;
@@ -212,8 +219,10 @@ __global__ void moe_combine_kernel(float* __restrict__ out, size_t ldo, const TY
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
         float total = 0.f;
         if (live) {
-            for (int j = 0; j < top; ++j)
-                total = fmaf(wts[t * top + j], to_f32(y[(size_t)pair_place[t * top + j] * ldy + d]), total);
+            for (int j = 0; j < top; ++j) {
+                const int place = pair_place[t * top + j];
+                total = fmaf(wts[t * top + j], place < n_rows ? to_f32(y[(size_t)place * ldy + d]) : load_as_f32(x, x_dtype, t * ldx + d), total);
+            }
             if (add) total = fmaf(load_as_f32(add, add_dtype, t * ldadd + d), add_scale ? add_scale[t] : 1.0f, total);
         }
         out[t * ldo + d] = total;
@@ -240,7 +249,7 @@ QS_API int qs_moe_route(int32_t* idx, float* wts, float* shared_gate, const floa
 
 QS_API int qs_moe_expert_up(void* hidden, long long ldh, const void* x, long long ldx, const void* w_up, int dtype,
                             const int32_t* idx, const int32_t* tok_slot, int T, int top, int D, int F, int act,
-                            int gated, cudaStream_t stream) {
+                            int gated, int n_experts, cudaStream_t stream) {
     if (T == 0) return QS_OK;
     QS_REQUIRE(T > 0 && top > 0 && D > 0 && F > 0, "moe_expert_up: bad sizes");
     QS_REQUIRE((size_t)D * sizeof(float) <= 200 * 1024, "moe_expert_up: width %d does not fit shared memory", D);
@@ -251,7 +260,7 @@ QS_API int qs_moe_expert_up(void* hidden, long long ldh, const void* x, long lon
     cudaError_t e = cudaSuccess;
 #define GO(TT) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_expert_up_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e == cudaSuccess) e = qs_launch_dependent(moe_expert_up_kernel<TT>, grid, dim3(256), smem, stream, (TT*)hidden, (size_t)ldh, (const TT*)x, \
-        (size_t)ldx, (const TT*)w_up, idx, tok_slot, top, D, F, rows_per_block, act, vec, gated); } while (0)
+        (size_t)ldx, (const TT*)w_up, idx, tok_slot, top, D, F, rows_per_block, act, vec, gated, n_experts); } while (0)
     if (dtype == QS_F32) GO(float);
     else if (dtype == QS_BF16) GO(__nv_bfloat16);
     else return qs_fail(QS_ERR_INVALID_INPUT, "moe_expert_up: unknown dtype %d", dtype);
@@ -262,7 +271,8 @@ QS_API int qs_moe_expert_up(void* hidden, long long ldh, const void* x, long lon
 
 QS_API int qs_moe_expert_down(float* out, long long ldo, const void* hidden, long long ldh, const void* w_down, int dtype,
                               const int32_t* idx, const float* wts, const int32_t* tok_slot, const void* add, int add_dtype,
-                              long long ldadd, const float* add_scale, int T, int top, int D, int F, cudaStream_t stream) {
+                              long long ldadd, const float* add_scale, int T, int top, int D, int F, const void* x, long long ldx,
+                              int n_experts, cudaStream_t stream) {
     if (T == 0) return QS_OK;
     QS_REQUIRE(T > 0 && top > 0 && D > 0 && F > 0, "moe_expert_down: bad sizes");
     const size_t smem = (size_t)top * F * sizeof(float);
@@ -273,7 +283,8 @@ QS_API int qs_moe_expert_down(float* out, long long ldo, const void* hidden, lon
     cudaError_t e = cudaSuccess;
 #define GO(TT) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(moe_expert_down_kernel<TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
     if (e == cudaSuccess) e = qs_launch_dependent(moe_expert_down_kernel<TT>, grid, dim3(256), smem, stream, out, (size_t)ldo, (const TT*)hidden, \
-        (size_t)ldh, (const TT*)w_down, idx, wts, tok_slot, add, add_dtype, (size_t)ldadd, add_scale, top, D, F, rows_per_block, vec); } while (0)
+        (size_t)ldh, (const TT*)w_down, idx, wts, tok_slot, add, add_dtype, (size_t)ldadd, add_scale, top, D, F, rows_per_block, vec, (const TT*)x, (size_t)ldx, \
+        n_experts); } while (0)
     if (dtype == QS_F32) GO(float);
     else if (dtype == QS_BF16) GO(__nv_bfloat16);
     else return qs_fail(QS_ERR_INVALID_INPUT, "moe_expert_down: unknown dtype %d", dtype);
@@ -291,13 +302,14 @@ QS_API int qs_moe_sort(int32_t* offsets, int32_t* place_token, int32_t* pair_pla
 
 QS_API int qs_moe_combine(float* out, long long ldo, const void* y, int y_dtype, long long ldy, const int32_t* pair_place,
                           const float* wts, const int32_t* tok_slot, const void* add, int add_dtype, long long ldadd,
-                          const float* add_scale, int T, int top, int D, cudaStream_t stream) {
+                          const float* add_scale, int T, int top, int D, const void* x, int x_dtype, long long ldx, int n_rows,
+                          cudaStream_t stream) {
     if (T == 0) return QS_OK;
     QS_REQUIRE(T > 0 && top > 0 && D > 0, "moe_combine: bad sizes");
     const int threads = D >= 1024 ? 256 : 128;
     cudaError_t e;
 #define GO(TY) e = qs_launch_dependent(moe_combine_kernel<TY>, dim3(T), dim3(threads), 0, stream, out, (size_t)ldo, (const TY*)y, \
-        (size_t)ldy, pair_place, wts, tok_slot, add, add_dtype, (size_t)ldadd, add_scale, top, D)
+        (size_t)ldy, pair_place, wts, tok_slot, add, add_dtype, (size_t)ldadd, add_scale, top, D, x, x_dtype, (size_t)ldx, n_rows)
     if (y_dtype == QS_F32) GO(float);
     else if (y_dtype == QS_BF16) GO(__nv_bfloat16);
     else return qs_fail(QS_ERR_INVALID_INPUT, "moe_combine: unknown dtype %d", y_dtype);

@@ -29,6 +29,7 @@ _SIGNATURES = {
                       c_longlong, c_longlong, c_int, c_void_p], c_int),
     "qs_gather_rows": ([c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_longlong, c_void_p], c_int),
     "qs_add": ([c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_void_p], c_int),
+    "qs_scale": ([c_void_p, c_longlong, c_float, c_void_p], c_int),
     "qs_linear_simt": ([c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p,
                         c_void_p, c_int, c_int, c_int, c_longlong, c_longlong, c_longlong, c_void_p], c_int),
     "qs_rope_store": ([c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_longlong,
@@ -37,6 +38,9 @@ _SIGNATURES = {
     "qs_norm_rope_store": ([c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_longlong, c_void_p, c_int, c_void_p, c_int,
                             c_float, c_int, c_int, c_int, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int,
                             c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p], c_int),
+    "qs_rope_unit_store": ([c_void_p, c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_longlong, c_float, c_int, c_int, c_int, c_int, c_int,
+                            c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int,
+                            c_void_p], c_int),
     "qs_attention": ([c_void_p, c_void_p, c_int, c_longlong, c_longlong, c_void_p, c_void_p, c_void_p, c_int,
                       c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p,
                       c_int, c_float, c_int, c_int, c_void_p, c_int, c_int, c_void_p], c_int),
@@ -76,6 +80,8 @@ _SIGNATURES = {
                         c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p], c_int),
     "qs_stream_tanh_norm": ([c_void_p, c_longlong, c_int, c_int, c_float, *([c_void_p, c_longlong, c_float, c_void_p, c_int] * 3), c_int,
                              *([c_void_p, c_longlong, c_float, c_void_p, c_int, c_void_p, c_int] * 2), c_void_p], c_int),
+    "qs_stream_norm": ([c_void_p, c_longlong, c_int, c_int, c_float, c_int, *([c_void_p, c_longlong, c_float] * 3), c_int, c_void_p, c_longlong,
+                        c_void_p, c_int, c_void_p, c_int, c_int, c_void_p], c_int),
     "qs_short_conv": ([c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_longlong,
                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p], c_int),
     "qs_conv_keep": ([c_void_p, c_longlong, c_void_p, c_longlong, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p], c_int),
@@ -98,12 +104,12 @@ _SIGNATURES = {
     "qs_moe_route": ([c_void_p, c_void_p, c_void_p, c_void_p, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_float, c_int, c_int, c_int, c_float, c_void_p], c_int),
     "qs_moe_expert_up": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_int, c_int,
-                          c_int, c_int, c_int, c_int, c_void_p], c_int),
+                          c_int, c_int, c_int, c_int, c_int, c_void_p], c_int),
     "qs_moe_expert_down": ([c_void_p, c_longlong, c_void_p, c_longlong, c_void_p, c_int, c_void_p, c_void_p, c_void_p,
-                            c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p], c_int),
+                            c_void_p, c_int, c_longlong, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_longlong, c_int, c_void_p], c_int),
     "qs_moe_sort": ([c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p], c_int),
     "qs_moe_combine": ([c_void_p, c_longlong, c_void_p, c_int, c_longlong, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
-                        c_longlong, c_void_p, c_int, c_int, c_int, c_void_p], c_int),
+                        c_longlong, c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_longlong, c_int, c_void_p], c_int),
     "qs_token_shift": ([c_void_p, c_longlong, c_longlong, c_void_p, c_longlong, c_int, c_void_p, c_void_p, c_longlong,
                         c_void_p, c_void_p, c_int, c_int, c_int, c_void_p], c_int),
     "qs_argmax": ([c_void_p, c_void_p, c_int, c_int, c_longlong, c_void_p], c_int),
@@ -263,6 +269,14 @@ def add(a: torch.Tensor, b: torch.Tensor, c=None) -> torch.Tensor:
     return out
 
 
+def scale(x: torch.Tensor, factor: float) -> torch.Tensor:
+    """x <- factor * x in place (contiguous float32)."""
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise QStreamError(QsError.INVALID_INPUT, "scale: need a contiguous float32 tensor")
+    check(library().qs_scale(ptr(x), x.numel(), float(factor), stream()))
+    return x
+
+
 def linear_simt(x, weight, bias=None, activation=None, residuals=(), out_dtype=None, out=None) -> torch.Tensor:
     """act(x W^T + bias) + residuals, accumulated in true 32-bit on the CUDA cores."""
     M, K, lda = _rows(x)
@@ -329,6 +343,22 @@ def norm_rope_store(q, k, v, q_weight, k_weight, eps, n_heads, n_kv_heads, head_
         _int32(page_table, "page_table") if page_table is not None else None,
         page_table.shape[1] if page_table is not None else 0, int(page_tokens), ptr(k_cache), ptr(v_cache), T, ptr(status),
         int(bool(half_layout)), stream()))
+
+
+def rope_unit_store(q, k, v, eps, n_heads, n_kv_heads, head_dim, rotary_dim, cos_sin, tok_slot, tok_pos, page_table, page_tokens, k_cache,
+                    v_cache, status, settled=False, v_head_dim=None, half_layout=False) -> None:
+    """The rotation of every head's first `rotary_dim` dims (none without `cos_sin`), then every head of q and k divided by its own
+    root mean square over head_dim (`eps` inside the root, no weight), then the cache write, in one kernel: q is changed in
+    place, the cache keeps the rotated and normed k and the values v as they are (v may be k: the keys as projected).
+    k = v = None (n_kv_heads = 0): queries only.  `settled`: as for `rope_store`."""
+    T = q.shape[0]
+    check(library().qs_rope_unit_store(
+        ptr(q), ptr(k), ptr(v), dtype_code(q), q.stride(0), k.stride(0) if k is not None else 0, v.stride(0) if v is not None else 0, float(eps),
+        int(n_heads), int(n_kv_heads) if k is not None else 0, int(head_dim), int(v_head_dim or head_dim),
+        int(rotary_dim) if cos_sin is not None else 0, ptr(cos_sin), cos_sin.shape[0] if cos_sin is not None else 0,
+        _int32(tok_slot, "tok_slot"), _int32(tok_pos, "tok_pos"), _int32(page_table, "page_table") if page_table is not None else None,
+        page_table.shape[1] if page_table is not None else 0, int(page_tokens), ptr(k_cache), ptr(v_cache), T, ptr(status),
+        int(bool(half_layout)), int(bool(settled)), stream()))
 
 
 def attention(q, n_heads, n_kv_heads, head_dim, scale, window, tok_slot, tok_pos, page_table,
@@ -473,12 +503,15 @@ def activate(x: torch.Tensor, activation) -> torch.Tensor:
     return x
 
 
-def gated_act(ab: torch.Tensor, activation) -> torch.Tensor:
-    """out = act(a) * b for ab = [a | b] ([rows, 2 F]), in 32-bit, rounded once."""
+def gated_act(ab: torch.Tensor, activation, out=None) -> torch.Tensor:
+    """out = act(a) * b for ab = [a | b] ([rows, 2 F]), in 32-bit, rounded once; `out`: an optional view with contiguous rows."""
     rows, two_f, ldi = _rows(ab)
     F = two_f // 2
-    out = torch.empty((rows, F), dtype=ab.dtype, device=ab.device)
-    check(library().qs_gated_act(ptr(out), F, ptr(ab), ldi, dtype_code(ab), rows, F, ACTIVATIONS[activation], stream()))
+    if out is None:
+        out = torch.empty((rows, F), dtype=ab.dtype, device=ab.device)
+    elif out.shape != (rows, F) or out.stride(1) != 1 or out.dtype != ab.dtype:
+        raise QStreamError(QsError.INVALID_INPUT, "gated_act: the output view does not fit")
+    check(library().qs_gated_act(ptr(out), out.stride(0), ptr(ab), ldi, dtype_code(ab), rows, F, ACTIVATIONS[activation], stream()))
     return out
 
 
@@ -716,6 +749,30 @@ def stream_tanh_norm(x, branches=(), eps: float = 0.0, reads=(), out_dtype=None)
     return hs
 
 
+def stream_norm(x, branches, weight, bias, eps: float, center: bool, out_dtype=None, settled=False) -> torch.Tensor:
+    """The 32-bit stream x [T, D] written and read in one pass.  `branches`: up to three (factor, y), y float32 [T, D] (a vector for
+    all tokens as a view whose rows are 0 apart): x <- x + sum of factor * y, in place.  Returns norm(x) * weight + bias (bias may
+    be None) of the new x in `out_dtype`: layer norm (`center`) or RMS norm, statistics in 32-bit, eps inside the root.
+    `settled`: as for `layernorm`."""
+    rows, D, ldx = _rows(x)
+    if x.dtype != torch.float32 or len(branches) > 3:
+        raise QStreamError(QsError.INVALID_INPUT, "stream_norm: a float32 stream and up to three branches")
+    if weight.numel() != D or (bias is not None and bias.numel() != D):
+        raise QStreamError(QsError.INVALID_INPUT, f"stream_norm: width {D} but weight {tuple(weight.shape)}")
+    args = []
+    for mult, y in [*branches, *[(0.0, None)] * (3 - len(branches))]:
+        ld = 0
+        if y is not None:
+            r2, D2, ld = _rows(y)
+            if (r2, D2) != (rows, D) or y.dtype != torch.float32:
+                raise QStreamError(QsError.INVALID_INPUT, "stream_norm: a branch differs from the stream in shape or type")
+        args += [ptr(y), ld, float(mult)]
+    h = torch.empty((rows, D), dtype=out_dtype or x.dtype, device=x.device)
+    check(library().qs_stream_norm(ptr(x), ldx, rows, D, float(eps), int(bool(center)), *args, dtype_code(h), ptr(h), h.stride(0), ptr(weight),
+                                   dtype_code(weight), ptr(bias), _code(bias), int(bool(settled)), stream()))
+    return h
+
+
 # ------------------------------------------------------------------------------- recurrences with a state per channel
 
 def short_conv(x, taps, bias, held, tok_slot, tok_pos, activation=None, decode=False) -> torch.Tensor:
@@ -907,7 +964,7 @@ def moe_experts_indirect(x, w_up, w_down, idx, wts, tok_slot, activation, add=No
     pair finds its expert's matrices (w_up [E, F, D], w_down [E, D, F]) on the device: for steps of few tokens.
     `glu` = (limit, alpha, shift): gated experts, w_up [E, 2 F, D] holding an expert's gate rows above its up rows; the
     hidden vector is `clamped_glu` of the two halves.  `gated`: w_up likewise, the hidden vector act(gate) * up, taken
-    inside the first kernel."""
+    inside the first kernel.  A choice idx >= E stands for an expert that returns x[t] itself."""
     T, D, ldx = _rows(x)
     E, F, _ = w_up.shape
     top = idx.shape[1]
@@ -918,13 +975,13 @@ def moe_experts_indirect(x, w_up, w_down, idx, wts, tok_slot, activation, add=No
     hidden = torch.empty((T * top, F), dtype=x.dtype, device=x.device)
     out = torch.empty((T, D), dtype=torch.float32, device=x.device)
     check(library().qs_moe_expert_up(ptr(hidden), F, ptr(x), ldx, ptr(w_up), dtype_code(x), _int32(idx, "idx"),
-                                     _int32(tok_slot, "tok_slot"), T, top, D, F, ACTIVATIONS[None if glu else activation], int(bool(gated)), stream()))
+                                     _int32(tok_slot, "tok_slot"), T, top, D, F, ACTIVATIONS[None if glu else activation], int(bool(gated)), E, stream()))
     if glu:
         hidden = clamped_glu(hidden, *glu)
         F = F // 2
     check(library().qs_moe_expert_down(ptr(out), D, ptr(hidden), F, ptr(w_down), dtype_code(x), _int32(idx, "idx"), ptr(wts),
                                        _int32(tok_slot, "tok_slot"), ptr(add), _code(add),
-                                       add.stride(0) if add is not None else 0, ptr(add_scale), T, top, D, F, stream()))
+                                       add.stride(0) if add is not None else 0, ptr(add_scale), T, top, D, F, ptr(x), ldx, E, stream()))
     return out
 
 
@@ -960,14 +1017,18 @@ def expert_products(out, x, w_all, offsets) -> None:
     check(rc)
 
 
-def moe_combine(y, pair_place, wts, tok_slot, add=None, add_scale=None) -> torch.Tensor:
-    """out[t] = sum_j wts[t, j] y[pair_place[t, j]] (+ add[t] * add_scale[t]) in float32."""
-    _, D, ldy = _rows(y)
+def moe_combine(y, pair_place, wts, tok_slot, add=None, add_scale=None, x=None) -> torch.Tensor:
+    """out[t] = sum_j wts[t, j] y[pair_place[t, j]] (+ add[t] * add_scale[t]) in float32.  With `x` [T, D] a place behind y's last
+    row stands for x[t] (an expert that returns its input)."""
+    n_rows, D, ldy = _rows(y)
+    if x is not None and (x.shape != (wts.shape[0], D) or x.stride(1) != 1):
+        raise QStreamError(QsError.INVALID_INPUT, "moe_combine: the tokens' inputs do not fit")
     T, top = wts.shape
     out = torch.empty((T, D), dtype=torch.float32, device=y.device)
     check(library().qs_moe_combine(ptr(out), D, ptr(y), dtype_code(y), ldy, ptr(pair_place), ptr(wts),
                                    _int32(tok_slot, "tok_slot"), ptr(add), _code(add), add.stride(0) if add is not None else 0,
-                                   ptr(add_scale), T, top, D, stream()))
+                                   ptr(add_scale), T, top, D, ptr(x), _code(x), x.stride(0) if x is not None else 0,
+                                   n_rows if x is not None else 2**31 - 1, stream()))
     return out
 
 

@@ -7,6 +7,9 @@
 //   stream_tanh_norm   x <- x + sum of up to three branches (32-bit, in place), each with a factor and, if it has a
 //                      weight, divided by its root mean square first; then up to two reads of the new x in the same
 //                      pass: tanh(alpha x) * w + b (no statistics), or x itself
+//   stream_norm        x <- x + sum of up to three branches (32-bit, in place), each with a factor (a branch whose rows
+//                      are 0 apart is one vector for all tokens), and h = norm(x) * w + b of the new x in the same pass, with
+//                      norm = layer norm or RMS norm
 //   gated_group_norm   out = o / sqrt(mean_group(o^2) + eps) * w * act(gate), groups of consecutive elements
 //                      (one group = the whole row, or one per head; group 0 = no norm, only the gate)
 //   gated_act          out = act(a) * b for the two halves [a | b] of a fused projection (gated feed-forward)
@@ -137,6 +140,20 @@ int launch_branch_norm(void* h_out, long long ldh, void* x, long long ldx, const
 
 // ----------------------------------------------------------------------------- branches into the stream, tanh norms
 
+// Four neighbouring elements of a vector or a row, as stored.
+template <typename T> struct FourOf;
+template <> struct FourOf<float> { typedef float4 type; };
+template <> struct FourOf<__nv_bfloat16> { typedef uint2 type; };
+__device__ __forceinline__ float4 four_as_f32(float4 v) { return v; }
+__device__ __forceinline__ float4 four_as_f32(uint2 v) {
+    return make_float4(__uint_as_float(v.x << 16), __uint_as_float(v.x & 0xffff0000u), __uint_as_float(v.y << 16), __uint_as_float(v.y & 0xffff0000u));
+}
+__device__ __forceinline__ void store_four(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
 struct StreamBranch { const float* y; size_t ld; const void* w; int w_dtype; float mult; };
 struct TanhRead { void* h; size_t ld; const void* w; const void* b; int w_dtype, b_dtype; float alpha; };
 
@@ -213,6 +230,112 @@ __global__ void stream_tanh_norm_kernel(float* __restrict__ x, size_t ldx, Strea
                 }
             }
     }
+}
+
+// ----------------------------------------------------------------------------- branches into the stream, one norm
+
+// One block per row; a thread holds PER pieces of four neighbouring columns in registers from the first load to the norm
+// (16-byte aligned rows of whole fours, D <= 4 * PER * threads).  `settled`: weight and bias were complete before the
+// previous kernel of the stream began; they are then fetched while that kernel still runs.
+template <typename TH, typename TW, int PER>
+__global__ void stream_norm_vec_kernel(float* __restrict__ x, size_t ldx, StreamBranch b0, StreamBranch b1, StreamBranch b2, TH* __restrict__ h,
+                                       size_t ldh, const TW* __restrict__ w, const TW* __restrict__ b, int D, float eps, int center, int settled) {
+    __shared__ float scratch[33];
+    grid_dep_launch();
+    if (!settled) grid_dep_wait();
+    typedef typename FourOf<TW>::type W4;
+    W4 wv[PER], bv[PER];
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+        if (c < D) {
+            wv[p] = *reinterpret_cast<const W4*>(w + c);
+            if (b) bv[p] = *reinterpret_cast<const W4*>(b + c);
+        }
+    }
+    if (settled) grid_dep_wait();
+    const size_t t = blockIdx.x;
+    float* xr = x + t * ldx;
+    float4 v[PER];
+    float s = 0.f;
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+        v[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (c < D) v[p] = *reinterpret_cast<const float4*>(xr + c);
+    }
+    if (b0.y) {
+        const StreamBranch br[3] = {b0, b1, b2};
+#pragma unroll
+        for (int k = 0; k < 3; ++k) {
+            if (!br[k].y) continue;
+            const float* yr = br[k].y + t * br[k].ld;
+            float4 y[PER];
+#pragma unroll
+            for (int p = 0; p < PER; ++p) {
+                const int c = (p * blockDim.x + threadIdx.x) * 4;
+                y[p] = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c < D) y[p] = *reinterpret_cast<const float4*>(yr + c);
+            }
+#pragma unroll
+            for (int p = 0; p < PER; ++p) {
+                v[p].x = fmaf(br[k].mult, y[p].x, v[p].x); v[p].y = fmaf(br[k].mult, y[p].y, v[p].y);
+                v[p].z = fmaf(br[k].mult, y[p].z, v[p].z); v[p].w = fmaf(br[k].mult, y[p].w, v[p].w);
+            }
+        }
+#pragma unroll
+        for (int p = 0; p < PER; ++p) {
+            const int c = (p * blockDim.x + threadIdx.x) * 4;
+            if (c < D) *reinterpret_cast<float4*>(xr + c) = v[p];
+        }
+    }
+    float mean = 0.f;
+    if (center) {
+#pragma unroll
+        for (int p = 0; p < PER; ++p) s += (v[p].x + v[p].y) + (v[p].z + v[p].w);
+        mean = block_sum(s, scratch) / (float)D;
+    }
+    float q = 0.f;
+#pragma unroll
+    for (int p = 0; p < PER; ++p)
+        if ((p * blockDim.x + threadIdx.x) * 4 < D) {
+            v[p].x -= mean; v[p].y -= mean; v[p].z -= mean; v[p].w -= mean;
+            q = fmaf(v[p].x, v[p].x, q); q = fmaf(v[p].y, v[p].y, q); q = fmaf(v[p].z, v[p].z, q); q = fmaf(v[p].w, v[p].w, q);
+        }
+    const float rstd = 1.0f / sqrtf(block_sum(q, scratch) / (float)D + eps);
+#pragma unroll
+    for (int p = 0; p < PER; ++p) {
+        const int c = (p * blockDim.x + threadIdx.x) * 4;
+        if (c >= D) continue;
+        const float4 wf = four_as_f32(wv[p]), bf = b ? four_as_f32(bv[p]) : make_float4(0.f, 0.f, 0.f, 0.f);
+        store_four(h + t * ldh + c, make_float4(fmaf(v[p].x * rstd, wf.x, bf.x), fmaf(v[p].y * rstd, wf.y, bf.y),
+                                                fmaf(v[p].z * rstd, wf.z, bf.z), fmaf(v[p].w * rstd, wf.w, bf.w)));
+    }
+}
+
+// The same for any width and alignment: the row in shared memory as 32-bit floats.
+template <typename TH>
+__global__ void stream_norm_kernel(float* __restrict__ x, size_t ldx, StreamBranch b0, StreamBranch b1, StreamBranch b2, TH* __restrict__ h, size_t ldh,
+                                   const void* __restrict__ w, int w_dtype, const void* __restrict__ b, int b_dtype, int D, float eps, int center) {
+    extern __shared__ float row[];
+    __shared__ float scratch[33];
+    grid_dep_launch();
+    grid_dep_wait();
+    const size_t t = blockIdx.x;
+    const StreamBranch br[3] = {b0, b1, b2};
+    for (int i = threadIdx.x; i < D; i += blockDim.x) {
+        float v = x[t * ldx + i];
+        if (b0.y) {
+#pragma unroll
+            for (int k = 0; k < 3; ++k)
+                if (br[k].y) v = fmaf(br[k].mult, br[k].y[t * br[k].ld + i], v);
+            x[t * ldx + i] = v;
+        }
+        row[i] = v;
+    }
+    const float2 st = row_statistic(row, D, eps, center, scratch);
+    for (int i = threadIdx.x; i < D; i += blockDim.x)
+        h[t * ldh + i] = from_f32<TH>(fmaf((row[i] - st.x) * st.y, load_as_f32(w, w_dtype, i), b ? load_as_f32(b, b_dtype, i) : 0.f));
 }
 
 // ----------------------------------------------------------------------------- gated group norm
@@ -465,6 +588,47 @@ QS_API int qs_stream_tanh_norm(float* x, long long ldx, int rows, int D, float e
 #undef GO
     if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "stream_tanh_norm: %s", cudaGetErrorString(e));
     return qs_check_launch("stream_tanh_norm");
+}
+
+// x [rows, D] float32 (row stride ldx).  Branches y0..y2 float32 or null (a null one ends the list), with factors m0..m2; a row
+// stride of 0 gives every row the same vector.  h [rows, D] of type `h_dtype` = norm(x) * w + b (b may be null); `center` != 0:
+// layer norm, 0: RMS norm; statistics in 32-bit, eps inside the root.
+QS_API int qs_stream_norm(float* x, long long ldx, int rows, int D, float eps, int center, const float* y0, long long ld0, float m0,
+                          const float* y1, long long ld1, float m1, const float* y2, long long ld2, float m2, int h_dtype, void* h,
+                          long long ldh, const void* w, int w_dtype, const void* b, int b_dtype, int settled, cudaStream_t stream) {
+    if (rows == 0) return QS_OK;
+    QS_REQUIRE(rows > 0 && D > 0 && x && h && w, "stream_norm: bad sizes");
+    QS_REQUIRE((y0 || !y1) && (y1 || !y2), "stream_norm: a branch behind a missing one");
+    QS_REQUIRE(h_dtype == QS_F32 || h_dtype == QS_BF16, "stream_norm: unknown dtype %d", h_dtype);
+    QS_REQUIRE((size_t)D * sizeof(float) <= 200 * 1024, "stream_norm: width %d does not fit one block's shared memory", D);
+    typedef __nv_bfloat16 bf16;
+    const StreamBranch b0 = {y0, (size_t)ld0, nullptr, 0, m0}, b1 = {y1, (size_t)ld1, nullptr, 0, m1}, b2 = {y2, (size_t)ld2, nullptr, 0, m2};
+    auto fits = [](const void* p, long long ld) { return !p || (((uintptr_t)p % 16) == 0 && ld % 4 == 0); };
+    const bool vec = D % 4 == 0 && D <= 16384 && fits(x, ldx) && fits(y0, ld0) && fits(y1, ld1) && fits(y2, ld2) && fits(h, ldh) && fits(w, 0) &&
+                     fits(b, 0) && (!b || b_dtype == w_dtype);
+    cudaError_t e = cudaSuccess;
+    if (vec) {
+        // many rows: few threads with several loads in flight each; few rows: as many threads as help
+        const int per = rows >= 256 ? (D >= 2048 ? 4 : (D >= 1024 ? 2 : 1)) : (D <= 2048 ? 1 : (D <= 4096 ? 2 : 4));
+        const int threads = ((D / 4 + per - 1) / per + 31) / 32 * 32;
+#define GOV(TH, TW, PER) e = qs_launch_dependent(stream_norm_vec_kernel<TH, TW, PER>, dim3(rows), dim3(threads), 0, stream, x, (size_t)ldx, b0, b1, b2, \
+        (TH*)h, (size_t)ldh, (const TW*)w, (const TW*)b, D, eps, center, settled)
+#define GOP(TH, TW) do { if (per == 1) GOV(TH, TW, 1); else if (per == 2) GOV(TH, TW, 2); else GOV(TH, TW, 4); } while (0)
+        if (h_dtype == QS_F32) { if (w_dtype == QS_F32) GOP(float, float); else GOP(float, bf16); }
+        else { if (w_dtype == QS_F32) GOP(bf16, float); else GOP(bf16, bf16); }
+#undef GOP
+#undef GOV
+    } else {
+        const size_t smem = (size_t)D * sizeof(float);
+        const int threads = D >= 4096 ? 512 : (D >= 1024 ? 256 : 128);
+#define GO(TH) do { if (smem > 48 * 1024) e = cudaFuncSetAttribute(stream_norm_kernel<TH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        if (e == cudaSuccess) e = qs_launch_dependent(stream_norm_kernel<TH>, dim3(rows), dim3(threads), smem, stream, x, (size_t)ldx, b0, b1, b2, \
+            (TH*)h, (size_t)ldh, w, w_dtype, b, b_dtype, D, eps, center); } while (0)
+        if (h_dtype == QS_F32) GO(float); else GO(bf16);
+#undef GO
+    }
+    if (e != cudaSuccess) return qs_fail(QS_ERR_INTERNAL, "stream_norm: %s", cudaGetErrorString(e));
+    return qs_check_launch("stream_norm");
 }
 
 QS_API int qs_gated_group_norm(void* out, int out_dtype, long long ldo, const void* o, int o_dtype, long long ldi,

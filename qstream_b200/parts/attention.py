@@ -14,7 +14,7 @@ product as q, k, v); keys seen
 only inside the query's chunk of positions, or inside a window that also keeps the sequence's first tokens; a learned
 sink per head in the softmax's denominator; two attention maps per head over the same values, joined as a difference
 with a unit RMS per head (differential attention); one RMS norm over the whole q and the whole k projection before the
-heads are split; values that are the keys as projected (no W_v); a sink of a fixed score without a tensor.
+heads are split, or a unit RMS per head behind the rotation; values that are the keys as projected (no W_v); a sink of a fixed score without a tensor.
 """
 from __future__ import annotations
 
@@ -45,7 +45,7 @@ class Attention(Mixer):
             d["k"] = TensorDecl((hkv, spec.width))
             if not getattr(spec, "values_from_keys", False):
                 d["v"] = TensorDecl((hv, spec.width))
-        if getattr(spec, "qk_norm", None):
+        if getattr(spec, "qk_norm", None) == "whole":
             d["q_norm"] = TensorDecl((hq,), "norm_weight")
             if not spec.shares_cache:
                 d["k_norm"] = TensorDecl((hkv,), "norm_weight")
@@ -74,8 +74,10 @@ class Attention(Mixer):
             raise QStreamError(QsError.INVALID_MODEL, f"attention: value_mix '{spec.value_mix}' does not fit")
         self.values_from_keys = bool(getattr(spec, "values_from_keys", False))
         self.qk_norm = getattr(spec, "qk_norm", None)
-        if self.qk_norm not in (None, "whole"):
+        if self.qk_norm not in (None, "whole", "head"):
             raise QStreamError(QsError.UNSUPPORTED_ARCH, f"attention: no norm of q and k of kind '{self.qk_norm}'")
+        if self.qk_norm == "head" and (getattr(spec, "maps", 1) > 1 or spec.value_mix):
+            raise QStreamError(QsError.UNSUPPORTED_ARCH, "attention: a norm per head with several maps or blended values")
         if self.values_from_keys and (spec.value_dim != getattr(spec, "maps", 1) * spec.head_dim or spec.value_mix or spec.qkv_bias):
             raise QStreamError(QsError.INVALID_MODEL, "attention: values taken from the keys have the keys' size, no bias and no blend")
         names = ["q"] if spec.shares_cache else (["q", "k"] if self.values_from_keys else ["q", "k", "v"])
@@ -109,8 +111,8 @@ class Attention(Mixer):
             if self.sink is not None:
                 raise QStreamError(QsError.INVALID_MODEL, "attention: a learned sink and a fixed one exclude each other")
             self.sink = torch.full((spec.n_heads,), float(spec.fixed_sink), dtype=torch.float32, device=runtime.device)
-        self.q_norm = tensors["q_norm"] if self.qk_norm else None
-        self.k_norm = tensors["k_norm"] if self.qk_norm and not spec.shares_cache else None
+        self.q_norm = tensors["q_norm"] if self.qk_norm == "whole" else None
+        self.k_norm = tensors["k_norm"] if self.qk_norm == "whole" and not spec.shares_cache else None
         # which of the kernels' options only the generic kernel offers
         self.masked = bool(self.chunk or self.keep_first or self.sink is not None or self.maps > 1)
         self.lam = 0.0
@@ -155,15 +157,26 @@ class Attention(Mixer):
         table = getattr(self.position, "fused_table", None) if self.position is not None else None
         # the norms over the whole q and k, the rotation and the cache write as one kernel (a rotation that offers no
         # table of angles: norms by themselves, then the rotation's own way)
-        fused_norm = bool(self.qk_norm) and (self.position is None or table is not None) and self.maps == 1 and not s.value_mix
-        if self.qk_norm and not fused_norm:             # one norm over all heads' rows at once, statistics in 32-bit
+        fused_norm = self.qk_norm == "whole" and (self.position is None or table is not None) and self.maps == 1 and not s.value_mix
+        if self.qk_norm == "whole" and not fused_norm:  # one norm over all heads' rows at once, statistics in 32-bit
             q = ops.rmsnorm(q, self.q_norm, float(s.eps), out_dtype=q.dtype)
         if s.gate and out is not None:
             raise QStreamError(QsError.INVALID_INPUT, "attention: a gated mixer writes its own output")
         half = bool(getattr(self.position, "half_layout", False))
         if self.maps > 1 and self.position is not None:
             raise QStreamError(QsError.UNSUPPORTED_ARCH, "attention: several maps per head with a rotation")
-        if fused_norm:
+        if self.qk_norm == "head":                      # rotation, a unit RMS per head and the cache write as one kernel
+            shares = s.shares_cache
+            k = None if shares else qkv[:, hq:hq + hkv]
+            v = None if shares else (k if self.values_from_keys else qkv[:, hq + hkv:hq + hkv + hv])
+            if self.position is not None and table is None:
+                if self.values_from_keys:
+                    v = v.clone()                       # the keys as projected, before they are rotated in place
+                self.position.apply(q, k, step, s.n_heads, s.n_kv_heads, s.head_dim)
+            ops.rope_unit_store(q, k, v, float(s.eps), s.n_heads, s.n_kv_heads, s.head_dim, getattr(self.position, "rotary_dim", 0) if table is not None else 0,
+                                table, b.tok_slot, b.tok_pos, view.page_table, view.page_tokens, None if shares else view.k,
+                                None if shares else view.v, step.status, settled=True, v_head_dim=s.value_dim, half_layout=half)
+        elif fused_norm:
             shares = s.shares_cache
             k = None if shares else qkv[:, hq:hq + hkv]
             v = None if shares else (k if self.values_from_keys else qkv[:, hq + hkv:hq + hkv + hv])
@@ -182,7 +195,7 @@ class Attention(Mixer):
         else:
             k = qkv[:, hq:hq + hkv]
             v = k if self.values_from_keys else qkv[:, hq + hkv:hq + hkv + hv]     # the keys as projected: the kernel only reads k
-            if self.qk_norm:
+            if self.qk_norm == "whole":
                 k = ops.rmsnorm(k, self.k_norm, float(s.eps), out_dtype=k.dtype)
             v_first = None
             if s.value_mix == "first":

@@ -383,6 +383,112 @@ class TwinNormBlock(Arrangement):
         return x
 
 
+class ScaledParallelBlock(Arrangement):
+    """One norm, both sublayers read it, and a factor on what they add: h = norm(x); x += m (mixer(h) + ffn(h)), with the
+    residual stream x in 32-bit whatever the engine's type and updated in place; a layer may have no feed-forward.  The branches
+    arrive in 32-bit from their last product and stay pending (`step.pending`): adding them to x and the next layer's norm
+    are one kernel (norms that offer `forward_branches`).
+
+    Where both parts end in a projection to the width (they offer `output_projection()` and `forward_hidden(..., out=view)`) and the
+    weights are bfloat16, a step with prompts runs the two projections as one matrix product over the concatenated hidden vectors.
+    In a decode step, whose kernels are short and wait for one another, the feed-forward runs whole on a second stream beside the
+    mixer: it reads nothing of the mixer's."""
+    norm_names = ("input",)
+    takes_pending = True
+
+    def __init__(self, spec, parts, runtime):
+        super().__init__(spec, parts, runtime)
+        import inspect
+        import torch
+        self.mult = float(spec.residual_scale)
+        self.wide = torch.float32
+        self._typed = {id(p): "out_dtype" in inspect.signature(p.forward).parameters for p in (self.mixer, self.ffn) if p}
+        self.fused_weight = None
+        if self.ffn is None or runtime.dtype != torch.bfloat16 or getattr(self.mixer.spec, "gate", False) \
+                or not all(hasattr(p, "output_projection") and hasattr(p, "forward_hidden") for p in (self.mixer, self.ffn)):
+            return
+        (wm, bm), (wf, bf) = self.mixer.output_projection(), self.ffn.output_projection()
+        if wm.dtype == wf.dtype == torch.bfloat16 and wm.shape[0] == wf.shape[0] and wm.shape[1] % 8 == 0 and wf.shape[1] % 8 == 0:
+            self.k_mixer = wm.shape[1]
+            self.fused_weight = torch.cat([wm, wf], dim=1).contiguous()
+            biases = [b.float() for b in (bm, bf) if b is not None]
+            self.fused_bias = sum(biases[1:], biases[0]) if biases else None
+            # the parts keep views of the fused matrix, so the weights are held once
+            self.mixer.w_out, self.ffn.down = self.fused_weight[:, :self.k_mixer], self.fused_weight[:, self.k_mixer:]
+
+    part_specs = classmethod(ScaledResidualBlock.part_specs.__func__)      # a layer may lack its feed-forward here too
+    build = classmethod(ScaledResidualBlock.build.__func__)
+
+    def cached_parts(self):
+        return getattr(self.mixer, "cached_parts", lambda: [self.mixer])()
+
+    def _branch(self, part, *args):
+        from ..csrc import ops
+        y = part.forward(*args, **({"out_dtype": self.wide} if self._typed[id(part)] else {}))
+        return (self.mult, y if y.dtype == self.wide else ops.convert(y, self.wide), None)
+
+    def _read(self, x, before):
+        norm = self.norms["input"]
+        if isinstance(before, PendingBranches) and hasattr(norm, "forward_branches") and all(w is None for _, _, w in before.branches):
+            return norm.forward_branches(x, [(c, y) for c, y, _ in before.branches])
+        return norm.forward(before.apply(x) if before is not None else x)
+
+    def forward(self, x, step, cache_id):
+        before, step.pending = step.pending, None
+        h = self._read(x, before)
+        if self.ffn is None:
+            ys = [self._branch(self.mixer, h, step, cache_id)]
+        elif step.batch.decode and getattr(step, "side_stream", None) is not None:
+            from .linear import beside_main_stream, shared_sms
+            with shared_sms() if h.shape[0] <= SHARED_SM_ROWS else contextlib.nullcontext():
+                with beside_main_stream(step.side_stream, h.device) as beside:
+                    ffn_branch = self._branch(self.ffn, h, step)
+                ys = [self._branch(self.mixer, h, step, cache_id), ffn_branch]
+                beside.join()
+        elif self.fused_weight is not None:
+            import torch
+            from .linear import linear
+            hidden = torch.empty((h.shape[0], self.fused_weight.shape[1]), dtype=h.dtype, device=h.device)
+            self.mixer.forward_hidden(h, step, cache_id, out=hidden[:, :self.k_mixer])
+            self.ffn.forward_hidden(h, step, out=hidden[:, self.k_mixer:])
+            ys = [(self.mult, linear(hidden, self.fused_weight, self.fused_bias, out_dtype=self.wide), None)]
+        else:
+            ys = [self._branch(self.mixer, h, step, cache_id), self._branch(self.ffn, h, step)]
+        step.pending = PendingBranches(ys, 0.0)
+        return x
+
+
+class LoopStep(Part):
+    """Before each pass of a looped group of layers: x <- x + step[t].  The vector joins the branches that are still to be added
+    to the stream, as one more of them (the same row for every token)."""
+    role = "joint"
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        from ..weights.loader import TensorDecl
+        return {"step": TensorDecl((spec.times, spec.width), "bias")}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.steps = [row.clone() for row in tensors["step"].float()]
+
+    def begin(self, x, step):
+        pass
+
+    def forward(self, x, step, t):
+        import torch
+        from ..csrc import ops
+        branches, eps = [], 0.0
+        if isinstance(step.pending, PendingBranches) and len(step.pending.branches) < 3:
+            branches, eps = list(step.pending.branches), step.pending.eps
+        else:
+            x = step.settle(x)
+        x = x if x.dtype == torch.float32 else ops.convert(x, torch.float32)
+        step.pending = PendingBranches([*branches, (1.0, self.steps[t].expand(x.shape[0], -1), None)], eps)
+        return x
+
+
 class LoopEntry(Part):
     """Before each pass of a looped group of layers: x <- W_in [x; x0] + step[t], x0 the embedding's output.  x (with what
     is still pending) and x0 lie side by side in one buffer in the engine's type, x0 written once a step; the product's
@@ -548,7 +654,9 @@ class HyperBlock(Arrangement):
 
 
 register("arrangement", "twin_norm", TwinNormBlock)
+register("arrangement", "scaled_parallel", ScaledParallelBlock)
 register("joint", "loop_entry", LoopEntry)
+register("joint", "loop_step", LoopStep)
 register("arrangement", "hyper", HyperBlock)
 register("connection", "hyper_connection", HyperConnection)
 register("arrangement", "parallel", ParallelBlock)

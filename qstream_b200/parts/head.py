@@ -1,9 +1,11 @@
 """Output head: logits = rows W^T + b in 32-bit, for the wanted rows only (QStream src/engine.c:1237-1241
-runs it for every token and drops the bias); `tied` takes the embedding table as W (:1200-1236)."""
+runs it for every token and drops the bias); `tied` takes the embedding table as W (:1200-1236).
+A factor on the logits is applied to the 32-bit result."""
 from __future__ import annotations
 
 import torch
 
+from ..csrc import ops
 from ..errors import QsError, QStreamError
 from ..weights.loader import TensorDecl
 from .base import Head, register
@@ -24,6 +26,7 @@ class LinearHead(Head):
         super().__init__(spec, tensors, runtime)
         self.weight = None if spec.tied else tensors["weight"]
         self.bias = tensors["bias"] if spec.bias else None
+        self.scale = float(getattr(spec, "scale", 1.0))
 
     def tie(self, embedding):
         weight = getattr(embedding, "weight", None)
@@ -32,7 +35,8 @@ class LinearHead(Head):
         self.weight = weight
 
     def forward(self, rows):
-        return linear(rows, self.weight, self.bias, out_dtype=torch.float32)
+        logits = linear(rows, self.weight, self.bias, out_dtype=torch.float32)
+        return logits if self.scale == 1.0 else ops.scale(logits, self.scale)
 
 
 register("head", "lm_head", LinearHead)

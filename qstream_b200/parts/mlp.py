@@ -71,8 +71,15 @@ class GatedMlp(FeedForward):
             self.down_bias = tensors["down_bias"]
 
     def forward(self, h, step, residuals=(), out_dtype=None):
-        g = ops.gated_act(linear(h, self.gate_up, self.gate_up_bias), self.spec.activation)
-        return linear(g, self.down, self.down_bias, residuals=residuals, out_dtype=out_dtype)
+        return linear(self.forward_hidden(h, step), self.down, self.down_bias, residuals=residuals, out_dtype=out_dtype)
+
+    # See Attention.output_projection: the same pair for a parallel block that fuses both projections.
+    def output_projection(self):
+        return self.down, self.down_bias
+
+    def forward_hidden(self, h, step, out=None):
+        """act(gate h) * (up h): [T, inner], written to `out` if given."""
+        return ops.gated_act(linear(h, self.gate_up, self.gate_up_bias), self.spec.activation, out=out)
 
 
 # A step of single tokens, or of at most this many rows, lets every (token, expert) pair find its expert's matrices
@@ -90,15 +97,17 @@ class RoutedExperts(FeedForward):
     expert, experts act(gate) * up (an expert's gate rows stacked above its up rows; the unit inside the first kernel where
     the pairs go through the routing table, a kernel of its own behind the products), and clamped gated experts
     (an expert's gate rows stacked above its up rows in one matrix; the clamped gated unit is a kernel of its own
-    between the two products)."""
+    between the two products), and `identity` more router outputs whose expert returns its input (the kernels that add a
+    token's results up read the input itself there)."""
     captures_any_step = False           # a step with many tokens reads the experts' row counts on the host
 
     @classmethod
     def declare(cls, spec):
-        d = {"router": TensorDecl((spec.n_experts, spec.width))}
+        outputs = spec.n_experts + getattr(spec, "identity", 0)
+        d = {"router": TensorDecl((outputs, spec.width))}
         gated = getattr(spec, "gated", False)
         if getattr(spec, "correction", True):
-            d["correction"] = TensorDecl((spec.n_experts,), "bias")
+            d["correction"] = TensorDecl((outputs,), "bias")
         for e in range(spec.n_experts):
             d[f"up{e}"], d[f"down{e}"] = TensorDecl((spec.inner, spec.width)), TensorDecl((spec.width, spec.inner))
             if gated:
@@ -118,6 +127,7 @@ class RoutedExperts(FeedForward):
         if spec.activation not in ops.ACTIVATIONS:
             raise QStreamError(QsError.UNSUPPORTED_ARCH, f"activation '{spec.activation}' has no kernel")
         E = spec.n_experts
+        self.outputs = E + int(getattr(spec, "identity", 0))            # what the router chooses among
         self.gated = getattr(spec, "gated", False)
         if self.gated not in (False, True, "act") or (self.gated == "act" and spec.shared_inner):
             raise QStreamError(QsError.UNSUPPORTED_ARCH, f"routed experts: gated '{self.gated}' with a shared expert of {spec.shared_inner}")
@@ -147,8 +157,8 @@ class RoutedExperts(FeedForward):
         import torch
         s, b = self.spec, step.batch
         z = linear(h, self.w_router, out_dtype=torch.float32)
-        idx, wts, gate = ops.moe_route(z, self.correction, s.n_experts, s.top, s.groups, s.keep, s.route_scale,
-                                       gate_col=s.n_experts if self.shared_gate else -1, scores=self.scores,
+        idx, wts, gate = ops.moe_route(z, self.correction, self.outputs, s.top, s.groups, s.keep, s.route_scale,
+                                       gate_col=self.outputs if self.shared_gate else -1, scores=self.scores,
                                        group_score=self.group_score, renorm_eps=self.renorm_eps)
         shared = None
         if self.shared and self.gated:
@@ -159,11 +169,12 @@ class RoutedExperts(FeedForward):
             out = ops.moe_experts_indirect(h, self.w_up, self.w_down, idx, wts, b.tok_slot, s.activation, shared, gate, glu=self.glu,
                                            gated=self.gated == "act")
         else:
-            offsets, place_token, pair_place = ops.moe_sort(idx, s.n_experts)
+            offsets, place_token, pair_place = ops.moe_sort(idx, self.outputs)
             rows = ops.gather_rows(h, place_token)
+            bounds = offsets.tolist()[:s.n_experts + 1]     # waits for the device: how many rows each expert got
+            rows = rows[:bounds[-1]]                        # behind them lie the pairs whose expert returns its input
             hidden = torch.empty((rows.shape[0], self.w_up.shape[1]), dtype=h.dtype, device=h.device)
             y = torch.empty((rows.shape[0], s.width), dtype=torch.float32, device=h.device)
-            bounds = offsets.tolist()                   # waits for the device: how many rows each expert got
             ops.expert_products(hidden, rows, self.w_up, bounds)        # a product per expert, launched by one call
             if self.gated == "act":
                 hidden = ops.gated_act(hidden, s.activation)            # one launch for all experts' rows
@@ -172,7 +183,7 @@ class RoutedExperts(FeedForward):
             else:
                 ops.activate(hidden, s.activation)
             ops.expert_products(y, hidden, self.w_down, bounds)
-            out = ops.moe_combine(y, pair_place, wts, b.tok_slot, shared, gate)
+            out = ops.moe_combine(y, pair_place, wts, b.tok_slot, shared, gate, x=h if self.outputs > s.n_experts else None)
         if residuals:
             raise QStreamError(QsError.INVALID_INPUT, "routed experts: residuals are added by the arrangement")
         return out if out_dtype in (None, torch.float32) else ops.convert(out, out_dtype)

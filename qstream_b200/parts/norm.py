@@ -93,6 +93,31 @@ class StreamNorm(Norm):
                                branch_weight=branch_norm.weight)
 
 
+class BranchSumNorm(Norm):
+    """A norm with a weight and perhaps a bias (layer norm if the spec says `center`, else RMS) that reads the 32-bit stream and
+    writes the engine's type.  `forward_branches` first adds branches (factor, y) to x, in place, in the same kernel."""
+    captures_any_step = True
+
+    @classmethod
+    def declare(cls, spec):
+        return {"weight": TensorDecl((spec.size,), "norm_weight"), **({"bias": TensorDecl((spec.size,), "bias")} if spec.bias else {})}
+
+    def __init__(self, spec, tensors, runtime):
+        super().__init__(spec, tensors, runtime)
+        self.weight, self.bias = tensors["weight"], tensors["bias"] if spec.bias else None
+        self.eps, self.center = float(spec.eps), bool(spec.center)
+
+    def forward(self, x):
+        import torch
+        if x.dtype != torch.float32:
+            x = ops.convert(x, torch.float32)
+        return self.forward_branches(x, ())
+
+    def forward_branches(self, x, branches):
+        """x <- x + sum of factor * y over the (factor, y) of `branches` (in place), then the norm of the new x."""
+        return ops.stream_norm(x, branches, self.weight, self.bias, self.eps, self.center, self.runtime.dtype, settled=True)
+
+
 class StreamSumNorm(Norm):
     """The RMS norm of the sum of a residual stream's copies: rows [n, streams * size] in 32-bit, the copies side by
     side; the result [n, size] in the engine's type."""
@@ -141,6 +166,7 @@ class TanhNorm(Norm):
 
 register("norm", "layernorm", LayerNorm)
 register("norm", "tanh_norm", TanhNorm)
+register("norm", "branch_sum_norm", BranchSumNorm)
 register("norm", "stream_sum_rmsnorm", StreamSumNorm)
 register("norm", "stream_norm", StreamNorm)
 register("norm", "rmsnorm", RmsNorm)
