@@ -5,7 +5,9 @@ the kernels that Fofinex adds (`bench.py --design fofinex`); and for a Sefuvik m
 (`bench.py --design sefuvik`); and for a Nutatar model beside a Fofinex model, the library's closest design (attention
 through a latent, routed experts, a matrix-state mixer, branches normed on their way into a 32-bit stream)
 (`bench.py --design nutatar`); and for a Fotanex model beside a Nutatar model, the closest again (softmax-routed gated
-experts, attention with sinks, linear recurrences, a 32-bit stream) (`bench.py --design fotanex`).
+experts, attention with sinks, linear recurrences, a 32-bit stream) (`bench.py --design fotanex`); and for a Vofinex model
+beside a Fotanex model, the closest (both sublayers on the same stream, chunked attention with sinks, softmax-routed gated
+experts, a loop) (`bench.py --design vofinex`).
 
 Sizes resemble a real model's layers: a width, heads of 128 (attention: a quarter as many key heads), a gated
 feed-forward of 8/3 width on every layer, the mixers in the order lightning, attention, lightning, wkv; the
@@ -132,6 +134,20 @@ def fotanex_config(width: int, layers: int) -> dict:
     }
     order = ["parallel", "rglru", "mamba2", "parallel"]
     return {"architecture": "Fotanex", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "layers": [kinds[order[i % 4]] for i in range(layers)],
+            "loop": {"start": 0, "stop": layers, "times": 1}, "max_positions": 8192}
+
+
+def vofinex_config(width: int, layers: int) -> dict:
+    """Heads of 128, a quarter as many key heads, chunks of 512, half of each head rotated; feed-forwards in turn dense (8/3 width) and
+    16 experts of a quarter width beside four router outputs that return their input, 4 per token; the layers form a loop that
+    runs once, so that a step enters it with its vector."""
+    heads = width // 128
+    ffs = ({"kind": "dense", "ff": (width * 8 // 3 + 255) // 256 * 256},
+           {"kind": "moe", "expert": {"ff": width // 4}, "router": {"experts": 16, "identity": 4, "top": 4}})
+    mixer = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 512},
+             "rot": {"dims": 64, "base": 10000.0}}
+    return {"architecture": "Vofinex", "vocab": VOCAB, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0}, "residual_mult": 0.5,
+            "logit_scale": 0.5, "layers": [{"type": "attention", "mixer": mixer, "mlp": ffs[i % 2]} for i in range(layers)],
             "loop": {"start": 0, "stop": layers, "times": 1}, "max_positions": 8192}
 
 
@@ -894,114 +910,141 @@ def kernel_table_fotanex(torch, np, pk, width=2048, T=4096, batch=32, ctx=2048):
     return rows
 
 
-def run_fotanex(args, pk) -> int:
-    import numpy as np
-    import torch
-    import qstream_b200 as qs
-    out = {"impl": "ours", "design": "fotanex", "beside": "nutatar", "dtype": "bf16", "data": "synthetic token ids, random weights",
-           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
-    for name, size in SIZES.items():
-        entry = {}
-        for which, cfg in (("fotanex", fotanex_config(**size)), ("nutatar", nutatar_config(**size))):
-            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
-            r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
-            r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
-            entry[which] = r
-            del model
-            torch.cuda.empty_cache()
-        out["sizes"][name] = entry
-    out["kernels"] = kernel_table_fotanex(torch, np, pk)
-    print(json.dumps(out))
-    return 0
+def kernel_table_vofinex(torch, np, pk, width=2048, T=4096, batch=32, ctx=2048):
+    """The kernels that Vofinex adds, each by itself beside the like kernel of the other designs: milliseconds and the
+    fraction of its roofline."""
+    from .csrc import attention_bf16, ops
+    from .parts.linear import linear
+    from .parts.rotary import _table
+    t = Timer(torch)
+    bf, f32 = torch.bfloat16, torch.float32
+    dev = "cuda"
+    H, d = width // 128, 128
+    G = max(1, H // 4)
+    hbm, tens = pk["hbm_gbs"] * 1e9, pk["bf16_tflops"] * 1e12
+    rows = []
+
+    def add(name, like, ms, nbytes=0, flops=0, bound="hbm"):
+        peak = {"hbm": hbm, "tensor": tens}[bound]
+        done = (nbytes if bound == "hbm" else flops) / (ms * 1e-3)
+        rows.append({"kernel": name, "like": like, "ms": round(ms, 4), "bound": bound, "frac": round(done / peak, 4)})
+
+    i32 = lambda a: torch.tensor(a, dtype=torch.int32, device=dev)          # noqa: E731
+    ff = (width * 8 // 3 + 255) // 256 * 256
+    for n, tag in ((T, "prompt"), (batch, "decode")):
+        x, w = torch.randn(n, width, device=dev), torch.randn(width, device=dev, dtype=bf)
+        ys, vec = [torch.randn(n, width, device=dev) for _ in range(3)], torch.randn(width, device=dev)
+        reads = [(0.5, w, w, None), (0.7, w, w, None)]
+        add(f"one branch joined, layer norm {tag}", "two branches joined, tanh norms",
+            t.kernel(lambda: ops.stream_norm(x, [(0.5, ys[0])], w, w, 1e-5, True, bf, settled=True)), n * width * 14)
+        add(f"two branches joined, layer norm {tag}", "two branches joined, tanh norms",
+            t.kernel(lambda: ops.stream_norm(x, [(0.5, ys[0]), (0.5, ys[1])], w, w, 1e-5, True, bf, settled=True)), n * width * 18)
+        add(f"two branches and a pass's vector joined, layer norm {tag}", "two branches joined, tanh norms",
+            t.kernel(lambda: ops.stream_norm(x, [(0.5, ys[0]), (0.5, ys[1]), (1.0, vec.expand(n, -1))], w, w, 1e-5, True, bf, settled=True)), n * width * 18)
+        add(f"two branches joined, one normed, two tanh norms {tag} (Fotanex)", "",
+            t.kernel(lambda: ops.stream_tanh_norm(x, [(0.5, ys[0], w), (1.0, ys[1], None)], 1e-5, reads, bf)), n * width * 20)
+        add(f"branch norm + update + read {tag} (Nutatar)", "",
+            t.kernel(lambda: ops.branch_norm(x, None, 1e-5, False, out_dtype=bf, branch=ys[0], branch_weight=w)), n * width * 14)
+        # a dense layer's two output projections as one product (prompts) or two (decode)
+        hidden, wf = torch.randn(n, H * d + ff, device=dev, dtype=bf), torch.randn(width, H * d + ff, device=dev, dtype=bf) * 0.02
+        for out_dtype, who in ((f32, ""), (bf, " with a bfloat16 result (GPT-J)")):
+            ms = t.kernel(lambda: linear(hidden, wf, out_dtype=out_dtype))
+            add(f"both output projections as one product {tag}{who}", "" if who else "the same with a bfloat16 result", ms, wf.numel() * 2,
+                2.0 * n * wf.numel(), "tensor" if tag == "prompt" else "hbm")
+        del x, ys, hidden
+    # rotation, a unit RMS per head, cache write
+    n_pages, tl, chunk = batch * ctx // 64, min(T, ctx), 512
+    table = torch.arange(n_pages, dtype=torch.int32, device=dev).view(batch, ctx // 64)
+    status = torch.zeros(1, dtype=torch.int32, device=dev)
+    kg, vg = (torch.randn(n_pages, G, 64, d, device=dev, dtype=bf) for _ in range(2))
+    angles = _table(64, 10000.0, 8192, dev)
+    wq, wk = torch.randn(H * d, device=dev, dtype=bf), torch.randn(G * d, device=dev, dtype=bf)
+    for n, tag, slot, pos in ((tl, "prompt", i32([0] * tl), i32(list(range(tl)))), (batch, "decode", i32(list(range(batch))), i32([ctx - 1] * batch))):
+        x = torch.randn(n, (H + 2 * G) * d, device=dev, dtype=bf)
+        q, k, v = x[:, :H * d], x[:, H * d:(H + G) * d], x[:, (H + G) * d:]
+        nbytes = n * (2 * H + 4 * G) * d * 2
+        add(f"rotation + unit RMS per head + cache write {tag}", "norms of q and k + rotation + cache write",
+            t.kernel(lambda: ops.rope_unit_store(q, k, v, 1e-5, H, G, d, 64, angles, slot, pos, table, 64, kg, vg, status, settled=True, half_layout=True)), nbytes)
+        add(f"norms of q and k + rotation + cache write {tag} (Nutatar)", "",
+            t.kernel(lambda: ops.norm_rope_store(q, k, v, wq, wk, 1e-5, H, G, d, 64, angles, slot, pos, table, 64, kg, vg, status, half_layout=True)), nbytes)
+        add(f"rotation by halves + cache write {tag} (Sefuvik)", "",
+            t.kernel(lambda: ops.rope_store(q, k, v, H, G, d, 64, angles, slot, pos, table, 64, kg, vg, status, settled=True, half_layout=True)),
+            n * (H + 4 * G) * d * 2)        # half of each query head is rotated
+    # attention in chunks with sinks (beside the same behind a gate)
+    dslot, dpos = i32(list(range(batch))), i32([ctx - 1] * batch)
+    tiles = torch.tensor([(s0, min(128, tl - s0), s0, 0) for s0 in range(0, tl, 128)][::-1], dtype=torch.int32, device=dev)
+    q, sink = torch.randn(tl, H * d, device=dev, dtype=bf), torch.randn(H, device=dev)
+    seen = sum(p % chunk + 1 for p in range(tl))
+    qd = q[:batch].contiguous()
+    for gate, who in ((None, ""), (torch.randn(tl, H, device=dev, dtype=bf), " behind a gate per head (Fotanex)")):
+        gd = gate[:batch].contiguous() if gate is not None else None
+        opts = dict(chunk=chunk, sink=sink, head_gate=gate is not None)
+        ms = t.kernel(lambda: attention_bf16.prefill(q, H, G, d, d ** -0.5, 0, tiles, table, 64, kg, vg, status, gate=gate, **opts))
+        add(f"attention in chunks of {chunk}, sinks, prompt {tl}{who}", "" if who else "the same behind a gate per head", ms, flops=4.0 * H * d * seen, bound="tensor")
+        ms = t.kernel(lambda: attention_bf16.decode(qd, H, G, d, d ** -0.5, 0, dslot, dpos, table, 64, kg, vg, ctx, status, gate=gd, **opts))
+        add(f"attention in chunks of {chunk}, sinks, decode {batch} x {ctx}{who}", "" if who else "the same behind a gate per head", ms,
+            batch * ((ctx - 1) % chunk + 1) * G * d * 4)
+    # routed experts, four of twenty outputs returning their input (beside sixteen experts and weights made to sum to one)
+    E, same, top, F = 16, 4, 4, width // 4
+    zr, corr = torch.randn(T, E + same, device=dev), torch.randn(E + same, device=dev) * 0.1
+    w_gu, w_down = torch.randn(E, 2 * F, width, device=dev, dtype=bf) * 0.02, torch.randn(E, width, F, device=dev, dtype=bf) * 0.02
+    h, slot_all = torch.randn(T, width, device=dev, dtype=bf), i32([0] * T)
+    for n_out, who in ((E + same, ""), (E, " (Fotanex)")):
+        def choose():
+            return ops.moe_route(zr, None if who else corr, n_out, top, 1, 1, 1.0, scores="softmax", group_score="max", renorm_eps=1e-20 if who else None)
+        add(f"router choice among {n_out}, prompt {T}{who}", "" if who else "router choice among 16", t.kernel(choose), T * (n_out + 2 * top) * 4)
+        idx, wts, _ = choose()
+        pairs = int((idx < E).sum())
+        for nb in (8, batch):
+            used = len(set(idx[:nb].flatten().tolist()) & set(range(E)))
+            ix, wt = idx[:nb].contiguous(), wts[:nb].contiguous()
+            ms = t.kernel(lambda: ops.moe_experts_indirect(h[:nb], w_gu, w_down, ix, wt, slot_all[:nb], "silu", gated=True))
+            add(f"gated experts through the routing table, {nb} tokens ({used} experts read){who}", "" if who else "without outputs that return their input",
+                ms, used * 3 * F * width * 2)
+
+        def grouped():
+            offsets, place_token, pair_place = ops.moe_sort(idx, n_out)
+            rows_ = ops.gather_rows(h, place_token)
+            bounds = offsets.tolist()[:E + 1]
+            rows_ = rows_[:bounds[-1]]
+            yy = torch.empty((rows_.shape[0], width), dtype=f32, device=dev)
+            hid = torch.empty((rows_.shape[0], 2 * F), dtype=bf, device=dev)
+            ops.expert_products(hid, rows_, w_gu, bounds)
+            ops.expert_products(yy, ops.gated_act(hid, "silu"), w_down, bounds)
+            return ops.moe_combine(yy, pair_place, wts, slot_all, x=None if who else h)
+        add(f"gated experts ordered by expert, {T} tokens ({pairs} pairs with matrices){who}", "" if who else "without outputs that return their input",
+            t.kernel(grouped, repeats=5), flops=6.0 * pairs * F * width, bound="tensor")
+    # the factor on the logits of a decode step
+    logits = torch.randn(batch, VOCAB, device=dev)
+    add(f"factor on the logits, decode {batch} x {VOCAB}", "", t.kernel(lambda: ops.scale(logits, 0.5)), logits.numel() * 8)
+    return rows
 
 
-def run_nutatar(args, pk) -> int:
-    import numpy as np
-    import torch
-    import qstream_b200 as qs
-    out = {"impl": "ours", "design": "nutatar", "beside": "fofinex", "dtype": "bf16", "data": "synthetic token ids, random weights",
-           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
-    for name, size in SIZES.items():
-        entry = {}
-        for which, cfg in (("nutatar", nutatar_config(**size)), ("fofinex", fofinex_config(**size))):
-            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
-            r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
-            r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
-            entry[which] = r
-            del model
-            torch.cuda.empty_cache()
-        out["sizes"][name] = entry
-    out["kernels"] = kernel_table_nutatar(torch, np, pk)
-    print(json.dumps(out))
-    return 0
-
-
-def run_fofinex(args, pk) -> int:
-    import numpy as np
-    import torch
-    import qstream_b200 as qs
-    out = {"impl": "ours", "design": "fofinex", "beside": "lutelorn", "dtype": "bf16", "data": "synthetic token ids, random weights",
-           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
-    for name, size in SIZES.items():
-        entry = {}
-        for which, cfg in (("fofinex", fofinex_config(**size)), ("lutelorn", lutelorn_config(**size))):
-            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
-            r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
-            r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
-            entry[which] = r
-            del model
-            torch.cuda.empty_cache()
-        out["sizes"][name] = entry
-    out["kernels"] = kernel_table_fofinex(torch, np, pk)
-    print(json.dumps(out))
-    return 0
-
-
-def run_sefuvik(args, pk) -> int:
-    import numpy as np
-    import torch
-    import qstream_b200 as qs
-    out = {"impl": "ours", "design": "sefuvik", "beside": "lutelorn", "dtype": "bf16", "data": "synthetic token ids, random weights",
-           "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
-    for name, size in SIZES.items():
-        entry = {}
-        for which, cfg in (("sefuvik", sefuvik_config(**size)), ("lutelorn", lutelorn_config(**size))):
-            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
-            r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
-            r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
-            entry[which] = r
-            del model
-            torch.cuda.empty_cache()
-        out["sizes"][name] = entry
-    out["kernels"] = kernel_table_sefuvik(torch, np, pk)
-    print(json.dumps(out))
-    return 0
+# design -> (the model beside it, the table of its kernels)
+DESIGNS = {"lutelorn": ("gptj", kernel_table), "fofinex": ("lutelorn", kernel_table_fofinex), "sefuvik": ("lutelorn", kernel_table_sefuvik),
+           "nutatar": ("fofinex", kernel_table_nutatar), "fotanex": ("nutatar", kernel_table_fotanex), "vofinex": ("fotanex", kernel_table_vofinex)}
+CONFIGS = {"gptj": gptj_config, "lutelorn": lutelorn_config, "fofinex": fofinex_config, "sefuvik": sefuvik_config, "nutatar": nutatar_config,
+           "fotanex": fotanex_config, "vofinex": vofinex_config}
 
 
 def run(args, pk) -> int:
-    if getattr(args, "design", "") == "fofinex":
-        return run_fofinex(args, pk)
-    if getattr(args, "design", "") == "sefuvik":
-        return run_sefuvik(args, pk)
-    if getattr(args, "design", "") == "nutatar":
-        return run_nutatar(args, pk)
-    if getattr(args, "design", "") == "fotanex":
-        return run_fotanex(args, pk)
     import numpy as np
     import torch
     import qstream_b200 as qs
-    out = {"impl": "ours", "design": "lutelorn", "beside": "gptj", "dtype": "bf16", "data": "synthetic token ids, random weights",
+    design = getattr(args, "design", "") or "lutelorn"
+    beside, table = DESIGNS[design]
+    out = {"impl": "ours", "design": design, "beside": beside, "dtype": "bf16", "data": "synthetic token ids, random weights",
            "peaks": {k: pk[k] for k in ("hbm_gbs", "bf16_tflops", "source")}, "sizes": {}}
     for name, size in SIZES.items():
         entry = {}
-        for which, cfg in (("lutelorn", lutelorn_config(**size)), ("gptj", gptj_config(**size))):
-            model = qs.CausalLM.random(qs.config_from_dict(cfg), seed=0, dtype="bfloat16", device="cuda:0")
+        for which in (design, beside):
+            model = qs.CausalLM.random(qs.config_from_dict(CONFIGS[which](**size)), seed=0, dtype="bfloat16", device="cuda:0")
             r = model_throughput(qs, torch, np, model, VOCAB, 2048, 8, 1024, min(args.steps, 32), max(3, min(args.warmup, 4)))
             r["weights_mb"] = round(model.weight_bytes / 2**20, 1)
             entry[which] = r
             del model
             torch.cuda.empty_cache()
         out["sizes"][name] = entry
-    out["kernels"] = kernel_table(torch, np, pk)
+    out["kernels"] = table(torch, np, pk)
     print(json.dumps(out))
     return 0

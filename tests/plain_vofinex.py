@@ -64,6 +64,20 @@ def visible_keys(n, size):
     return (j <= i) & ((i // size == j // size) if size else True)
 
 
+def attend(q, k, v, scale, sink, visible):
+    """Softmax attention of q [T, H, d] over k [T, G, d] and v [T, G, dv] (query head h reads key head h // (H / G)), exp(sink[h])
+    one more term of the denominator: [T, H, dv]."""
+    T, H, G = q.shape[0], q.shape[1], k.shape[1]
+    out = np.zeros((T, H, v.shape[2]))
+    for hh in range(H):
+        g = hh // (H // G)
+        s = np.where(visible, (q[:, hh] @ k[:, g].T) * scale, -np.inf)
+        top = np.maximum(s.max(-1, keepdims=True), sink[hh])
+        e = np.exp(s - top)
+        out[:, hh] = (e / (e.sum(-1, keepdims=True) + np.exp(sink[hh] - top))) @ v[:, g]
+    return out
+
+
 def attention(m, w, p, h, eps):
     """Grouped softmax attention inside chunks of positions, with a learned sink per head in the denominator."""
     T = h.shape[0]
@@ -71,15 +85,7 @@ def attention(m, w, p, h, eps):
     G, dv = m.get("kv_heads", H), m.get("vdim", d)
     q, k = queries_and_keys(m, (h @ w[p + "q"].T).reshape(T, H, d), (h @ w[p + "k"].T).reshape(T, G, d), np.arange(T), eps)
     v = (h @ w[p + "v"].T).reshape(T, G, dv)
-    visible = visible_keys(T, (m.get("mask") or {}).get("size", 0))
-    out = np.zeros((T, H, dv))
-    for hh in range(H):
-        g = hh // (H // G)
-        s = np.where(visible, (q[:, hh] @ k[:, g].T) * m["scale"], -np.inf)
-        sink = float(w[p + "sink"][hh])
-        top = np.maximum(s.max(-1, keepdims=True), sink)
-        e = np.exp(s - top)
-        out[:, hh] = (e / (e.sum(-1, keepdims=True) + np.exp(sink - top))) @ v[:, g]
+    out = attend(q, k, v, m["scale"], w[p + "sink"], visible_keys(T, (m.get("mask") or {}).get("size", 0)))
     return out.reshape(T, H * dv) @ w[p + "o"].T
 
 
